@@ -12,379 +12,13 @@
 // launch_prefill_float).
 //
 // Every mbarrier wait is bounded (mq_device.cuh) and TMEM is always freed.
-#include <cuda.h>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
 
-#include <mutex>
-#include <unordered_map>
-
-#include "mq_device.cuh"
+#include "tc_attention.cuh"
 
 namespace mq {
-
-// ---------------------------------------------------------------- tcgen05 / TMA primitives
-__device__ __forceinline__ void tma_load_2d(void* smem_dst, const CUtensorMap* map, int x, int y, uint64_t* bar) {
-    asm volatile(
-        "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
-        ::"r"(smem_u32(smem_dst)), "l"(map), "r"(x), "r"(y), "r"(smem_u32(bar))
-        : "memory");
-}
-__device__ __forceinline__ void tma_load_3d(void* smem_dst, const CUtensorMap* map, int x, int y, int z, uint64_t* bar) {
-    asm volatile(
-        "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
-        ::"r"(smem_u32(smem_dst)), "l"(map), "r"(x), "r"(y), "r"(z), "r"(smem_u32(bar))
-        : "memory");
-}
-__device__ __forceinline__ void tmem_alloc(uint32_t* slot_smem, uint32_t ncols) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(slot_smem)), "r"(ncols) : "memory");
-    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
-}
-__device__ __forceinline__ void tmem_dealloc(uint32_t taddr, uint32_t ncols) {
-    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(taddr), "r"(ncols) : "memory");
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void umma_bf16(uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
-    asm volatile(
-        "{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-        ::"r"(d_tmem), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
-        : "memory");
-}
-// the same with the A operand in tensor memory (row i of A in lane i, two consecutive K elements per 32-bit column)
-__device__ __forceinline__ void umma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
-    asm volatile(
-        "{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
-        ::"r"(d_tmem), "r"(a_tmem), "l"(bdesc), "r"(idesc), "r"(accumulate)
-        : "memory");
-}
-// arrive on `bar` once every MMA issued so far by this thread has completed
-__device__ __forceinline__ void umma_commit(uint64_t* bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-        "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
-        "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];"
-        : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),
-          "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]),
-          "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]),
-          "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-        : "r"(taddr)
-        : "memory");
-    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-}
-
-__device__ __forceinline__ void tmem_ld32_nowait(uint32_t taddr, uint32_t (&r)[32]) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-        "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
-        "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];"
-        : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),
-          "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]),
-          "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]),
-          "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-        : "r"(taddr)
-        : "memory");
-}
-__device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
-__device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t (&r)[32]) {
-    asm volatile(
-        "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-        "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, "
-        "%17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31, %32};"
-        ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
-          "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]),
-          "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]),
-          "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
-        : "memory");
-    asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
-}
-
-// Shared-memory matrix descriptor of a K-major bf16 tile whose rows are 128 bytes
-// (64 elements) under the 128-byte swizzle: 8-row groups are 1024 bytes apart.
-__device__ __forceinline__ uint64_t smem_desc_sw128(const void* tile) {
-    uint64_t d = (uint64_t)((smem_u32(tile) >> 4) & 0x3fffu);
-    d |= 1ull << 16;                 // leading byte offset (unused for swizzled K-major), 16 B units
-    d |= (uint64_t)(1024 >> 4) << 32;  // stride byte offset between 8-row groups
-    d |= 1ull << 46;                 // descriptor version (sm_100)
-    d |= 2ull << 61;                 // SWIZZLE_128B
-    return d;
-}
-
-// The same tile read as an MN-major operand: [rows = K index][64 elements of the M / N dimension], i.e. a
-// row-major [k][n] matrix used as B without transposing it.  A 128-byte row holds 64 consecutive n of one k;
-// eight k form a 1024-byte swizzle group (stride byte offset); the next 64 n start panel_bytes further on
-// (leading byte offset).  A K = 16 step advances the start address by two groups.
-__device__ __forceinline__ uint64_t smem_desc_mn_sw128(const void* tile, uint32_t panel_bytes) {
-    uint64_t d = (uint64_t)((smem_u32(tile) >> 4) & 0x3fffu);
-    d |= (uint64_t)((panel_bytes >> 4) & 0x3fffu) << 16;
-    d |= (uint64_t)(1024 >> 4) << 32;
-    d |= 1ull << 46;
-    d |= 2ull << 61;
-    return d;
-}
-
-// Bounded wait that does not look at the sticky status word: used while a CTA drains after one of its
-// waits has expired (copies already issued must land, MMAs already issued must finish, before the CTA
-// hands back its shared and tensor memory).  About 1 ms.
-__device__ __forceinline__ bool mbar_wait_drain(uint64_t* bar, uint32_t parity) {
-    const long long t0 = clock64();
-    while (!mbar_try_wait(bar, parity))
-        if (clock64() - t0 > 2000000LL) return false;
-    return true;
-}
-
-// ---------------------------------------------------------------- GEMM  C[M,N] = A[M,K] * B[N,K]^T
-constexpr int GM_BM = 128;
-constexpr int GM_BK = 64;
-constexpr int GM_THREADS = 192;    // skinny GEMM: warp 0 TMA, warp 1 MMA + TMEM owner, warps 2..5 epilogue
-// Tile GEMM: eight epilogue warps.  Warps w and w + 4 read the same quarter of the TMEM lanes (a warp may
-// only touch lanes 32 (w % 4) .. + 31) and split the accumulator columns; with four warps the SwiGLU
-// epilogue of a 256 x 256 tile (65 536 silu + products on 128 threads) took as long as its main loop.
-constexpr int GM_EPI_WARPS = 8;
-constexpr int GM_TILE_THREADS = 64 + 32 * GM_EPI_WARPS;
-enum { EPI_STORE = 0, EPI_RESID = 1, EPI_SWIGLU = 2, EPI_PARTIAL = 3, EPI_STORE_2CTA = 4 };   // PARTIAL: fp32 plane blockIdx.z of a K split
-// EPI_STORE_2CTA: EPI_STORE with a three-stage ring (97 KB), so that two CTAs share an SM.  For a GEMM of many short
-// CTAs that stream weights (the batched LM head: 1187 column tiles of a 64-row matrix), where a lone CTA's start-up and
-// epilogue leave the SM's memory pipeline idle.
-
-// Every kernel of the prefill and batched-decode chains is launched with programmatic
-// stream serialisation and begins with griddepcontrol.wait + launch_dependents: the next
-// kernel's CTAs are scheduled (parameters loaded, shared memory carved) while this one runs,
-// which takes the launch latency of the ~230 (prefill) / ~310 (batched step) kernels of a
-// pass off the critical path.  Without the launch attribute both instructions are no-ops.
-template <typename... KArgs, typename... Args>
-static void launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args... args) {
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = grid;
-    cfg.blockDim = block;
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = stream;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = attr;
-    cfg.numAttrs = 1;
-    (void)cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);   // errors are sticky: callers read cudaGetLastError()
-}
-
-#ifndef MQ_GEMM_BUDGET_KB
-#define MQ_GEMM_BUDGET_KB 200   // shared memory for the operand ring of one CTA
-#define MQ_GEMM_MIN_CTAS 1
-#endif
-// MT = 128-row A tiles per CTA.  With MT = 2 a CTA computes a 256-row output tile with two
-// accumulators that share every B tile: the 128 x 128 tiles are bound by the operand traffic
-// from the L2 into the SMs, and a 256-row tile moves a third less of it per FLOP.
-template <int BN, int EPI, int MT = 1>
-struct GemmCfg {
-    static constexpr int NB = (EPI == EPI_SWIGLU) ? 2 : 1;                       // B operands per stage
-    static constexpr int A_BYTES = MT * GM_BM * GM_BK * 2;
-    static constexpr int STAGE_BYTES = A_BYTES + NB * BN * GM_BK * 2;
-    static constexpr int STAGES = EPI == EPI_STORE_2CTA ? 3 : (MQ_GEMM_BUDGET_KB * 1024) / STAGE_BYTES > 6 ? 6 : (MQ_GEMM_BUDGET_KB * 1024) / STAGE_BYTES;
-    static constexpr int ACC_COLS = MT * NB * BN;                                // accumulator columns in use
-    static constexpr int TMEM_COLS = ACC_COLS <= 32 ? 32 : ACC_COLS <= 64 ? 64 : ACC_COLS <= 128 ? 128 : ACC_COLS <= 256 ? 256 : 512;   // allocations are powers of two
-    static_assert(ACC_COLS <= 512 && BN % 32 == 0, "tensor memory holds 512 columns; the epilogue reads 32 at a time");
-    static constexpr size_t SMEM = (size_t)STAGES * STAGE_BYTES + 1024 /*align*/ + 256 /*barriers*/;
-};
-
-// x / (1 + e^-x) with the hardware exponential and reciprocal (2 ulp of fp32; the result is rounded to bf16)
-__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
-
-template <int BN, int EPI, int MT>
-__global__ void __launch_bounds__(GM_TILE_THREADS, MQ_GEMM_MIN_CTAS)
-k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const __grid_constant__ CUtensorMap tmB2,
-       const __grid_constant__ CUtensorMap tmB3, int tiles0, int tiles1,
-       bf16* __restrict__ C, const bf16* R, int M, int N, int K, int ldc, unsigned int* status, int drop_kb, int early_b) {
-    // drop_kb >= 0 (test hook): the producer never requests k-block drop_kb, so the MMA thread's wait for it
-    // runs out; -1 in every production launch.  early_b: B is constant over the stream's lifetime (a weight),
-    // so its first tiles may be requested before the preceding grid has finished.
-    pdl_trigger();   // the next grid may be scheduled already; it waits for this one below, after its own set-up
-    // EPI_STORE / EPI_RESID may concatenate up to three B matrices along N (q|k|v): column tile
-    // blockIdx.x < tiles0 reads tmB, < tiles0 + tiles1 tmB2, else tmB3.  EPI_SWIGLU uses tmB (gate)
-    // and tmB2 (up) for the same tile.
-    using Cfg = GemmCfg<BN, EPI, MT>;
-    extern __shared__ uint8_t smem_raw[];
-    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-    uint64_t* full = reinterpret_cast<uint64_t*>(smem + (size_t)Cfg::STAGES * Cfg::STAGE_BYTES);
-    uint64_t* empty = full + Cfg::STAGES;
-    uint64_t* accum = empty + Cfg::STAGES;
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(accum + 1);
-    // Set by the thread whose bounded wait expired (the sticky status bit is then set as well).  Everybody
-    // stops issuing work; the epilogue stores nothing; the CTA drains what is in flight before it exits.
-    volatile uint32_t* aborted = tmem_slot + 1;
-
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int m0 = blockIdx.y * GM_BM * MT, n0 = blockIdx.x * BN;
-    // EPI_PARTIAL: gridDim.z CTAs share an output tile, each takes a contiguous range of k-blocks
-    const int kb_first = (int)(((long long)blockIdx.z * (K / GM_BK)) / gridDim.z);
-    const int nk = (int)(((long long)(blockIdx.z + 1) * (K / GM_BK)) / gridDim.z) - kb_first;
-    const int tile = blockIdx.x;
-    const CUtensorMap* mapB = &tmB;
-    int brow0 = n0;
-    if (EPI != EPI_SWIGLU && tile >= tiles0) {
-        mapB = tile < tiles0 + tiles1 ? &tmB2 : &tmB3;
-        brow0 = (tile < tiles0 + tiles1 ? tile - tiles0 : tile - tiles0 - tiles1) * BN;
-    }
-
-    if (tid == 0) {
-        for (int s = 0; s < Cfg::STAGES; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
-        mbar_init(accum, 1);
-        mbar_fence_init();
-    }
-    if (tid == 64) *aborted = 0u;       // by a thread that is idle now (thread 0's set-up gates the first TMA request)
-    if (warp == 1) tmem_alloc(tmem_slot, Cfg::TMEM_COLS);
-    tc_fence_before();
-    __syncthreads();
-    tc_fence_after();
-    const uint32_t tmem_base = *reinterpret_cast<volatile uint32_t*>(tmem_slot);
-    // Barriers and tensor memory are set up while the preceding grid may still be running.  Where the B operand is
-    // a weight matrix that nothing on the stream writes, its tiles for the first ring of stages are requested now
-    // and cross HBM while that grid finishes; the A tiles (its output) follow the wait, from which on its results
-    // are complete and visible.
-    const int npre = !early_b ? 0 : nk < Cfg::STAGES ? nk : Cfg::STAGES;
-    if (tid == 0) {
-        for (int kb = 0; kb < npre; ++kb) {
-            if (kb == drop_kb) continue;
-            uint8_t* st = smem + (size_t)kb * Cfg::STAGE_BYTES;
-            mbar_expect_tx(&full[kb], (uint32_t)Cfg::STAGE_BYTES);
-            tma_load_2d(st + Cfg::A_BYTES, mapB, (kb_first + kb) * GM_BK, brow0, &full[kb]);
-            if (EPI == EPI_SWIGLU) tma_load_2d(st + Cfg::A_BYTES + BN * GM_BK * 2, &tmB2, (kb_first + kb) * GM_BK, n0, &full[kb]);
-        }
-    }
-    pdl_wait();
-
-    int issued = npre;                    // k-blocks the producer has requested, B tiles at least (thread 0 only)
-    if (warp == 0) {
-        if (lane == 0) {
-            for (int kb = 0; kb < nk; ++kb) {
-                const int s = kb % Cfg::STAGES;
-                if (kb >= Cfg::STAGES && !mbar_wait(&empty[s], (uint32_t)((kb / Cfg::STAGES) - 1) & 1u, status)) { *aborted = 1u; break; }
-                if (*aborted) break;
-                issued = kb + 1;
-                if (kb == drop_kb) continue;
-                uint8_t* st = smem + (size_t)s * Cfg::STAGE_BYTES;
-                if (kb >= npre) mbar_expect_tx(&full[s], (uint32_t)Cfg::STAGE_BYTES);
-#pragma unroll
-                for (int mt = 0; mt < MT; ++mt) tma_load_2d(st + mt * GM_BM * GM_BK * 2, &tmA, (kb_first + kb) * GM_BK, m0 + mt * GM_BM, &full[s]);
-                if (kb >= npre) {
-                    tma_load_2d(st + Cfg::A_BYTES, mapB, (kb_first + kb) * GM_BK, brow0, &full[s]);
-                    if (EPI == EPI_SWIGLU) tma_load_2d(st + Cfg::A_BYTES + BN * GM_BK * 2, &tmB2, (kb_first + kb) * GM_BK, n0, &full[s]);
-                }
-            }
-        }
-        __syncwarp();
-    } else if (warp == 1) {
-        if (lane == 0) {
-            // instruction descriptor: D = f32, A = B = bf16, both K-major, N >> 3, M >> 4.  EPI_SWIGLU: the gate
-            // and the up tile sit back to back in the stage (2 BN rows of one K-major operand), so ONE
-            // instruction of N = 2 BN fills both accumulators (columns [0, BN) gate, [BN, 2 BN) up).  A
-            // 128 x 128 x 16 instruction reads 8 KB of shared memory for 64 cycles of math, which is the
-            // SM's whole shared-memory bandwidth; at N = 256 it is 12 KB for 128 cycles.
-            constexpr int UMMA_N = Cfg::NB * BN;
-            static_assert(UMMA_N <= 256, "one instruction spans at most 256 columns");
-            const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(UMMA_N >> 3) << 17) | ((uint32_t)(GM_BM >> 4) << 24);
-            for (int kb = 0; kb < nk; ++kb) {
-                const int s = kb % Cfg::STAGES;
-                if (!mbar_wait(&full[s], (uint32_t)(kb / Cfg::STAGES) & 1u, status)) { *aborted = 1u; break; }
-                tc_fence_after();
-                uint8_t* st = smem + (size_t)s * Cfg::STAGE_BYTES;
-                const uint64_t db = smem_desc_sw128(st + Cfg::A_BYTES);
-#pragma unroll
-                for (int mt = 0; mt < MT; ++mt) {   // accumulator (mt, nb) lives at TMEM column (mt * NB + nb) * BN
-                    const uint64_t da = smem_desc_sw128(st + mt * GM_BM * GM_BK * 2);
-#pragma unroll
-                    for (int k = 0; k < GM_BK / 16; ++k) {
-                        const uint32_t acc = (kb > 0 || k > 0) ? 1u : 0u;
-                        umma_bf16(tmem_base + mt * Cfg::NB * BN, da + 2 * k, db + 2 * k, idesc, acc);   // +32 bytes per K=16 step
-                    }
-                }
-                umma_commit(&empty[s]);     // frees this stage once the MMAs above have read it
-            }
-            umma_commit(accum);             // accumulator complete (or, after an expired wait, the MMAs issued so far)
-            if (*aborted) mbar_wait_drain(accum, 0);   // tensor memory is freed below: nothing may still be writing it
-        }
-        __syncwarp();
-    } else {
-        // epilogue: warp (2..9) owns TMEM lanes 32*(warp%4) .. +31 = tile rows and half of the columns
-        const bool acc_ok = mbar_wait(accum, 0, status) && !*aborted;   // after an expired wait nothing is read or stored
-        tc_fence_after();
-        const int quarter = warp & 3, half = (warp - 2) >> 2;
-        // the two warps of a quarter take one 128-row accumulator each (MT = 2) or half of the columns (MT = 1)
-        static_assert(GM_EPI_WARPS == 8 && (MT == 2 || (BN / 2) % 32 == 0), "epilogue split");
-        const int cbeg = MT == 2 ? 0 : half * (BN / 2), cend = MT == 2 ? BN : cbeg + BN / 2;
-#pragma unroll 1
-        for (int mt = (MT == 2 ? half : 0); mt < (MT == 2 ? half + 1 : 1); ++mt) {
-        if (!acc_ok) break;
-        const int row = m0 + mt * GM_BM + quarter * 32 + lane;
-        const uint32_t trow = tmem_base + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(mt * Cfg::NB * BN);
-#pragma unroll 1
-        for (int c0 = cbeg; c0 < cend; c0 += 32) {
-            uint32_t v[32];
-            tmem_ld32(trow + c0, v);
-            if (EPI == EPI_PARTIAL) {   // raw fp32 accumulators into plane blockIdx.z of C (a float [gridDim.z][M][ldc] array)
-                if (row < M) {
-                    float4* fp = reinterpret_cast<float4*>(reinterpret_cast<float*>(C) + ((size_t)blockIdx.z * M + row) * ldc + n0 + c0);
-#pragma unroll
-                    for (int q = 0; q < 8; ++q)
-                        fp[q] = make_float4(__uint_as_float(v[4 * q]), __uint_as_float(v[4 * q + 1]), __uint_as_float(v[4 * q + 2]), __uint_as_float(v[4 * q + 3]));
-                }
-                continue;
-            }
-            uint32_t out[16];
-            if (EPI == EPI_SWIGLU) {
-                uint32_t u[32];
-                tmem_ld32(trow + BN + c0, u);
-#pragma unroll
-                for (int j = 0; j < 16; ++j) {
-                    const float g0 = rbf(__uint_as_float(v[2 * j])), g1 = rbf(__uint_as_float(v[2 * j + 1]));
-                    const float u0 = rbf(__uint_as_float(u[2 * j])), u1 = rbf(__uint_as_float(u[2 * j + 1]));
-                    out[j] = pack_bf16x2(rbf(silu_fast(g0)) * u0, rbf(silu_fast(g1)) * u1);
-                }
-            } else if (EPI == EPI_RESID) {
-                if (row < M) {
-                    const uint4* rp = reinterpret_cast<const uint4*>(R + (size_t)row * ldc + n0 + c0);
-#pragma unroll
-                    for (int q = 0; q < 4; ++q) {
-                        const uint4 rr = rp[q];
-                        const uint32_t rw[4] = {rr.x, rr.y, rr.z, rr.w};
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            const int j = q * 4 + e;
-                            out[j] = pack_bf16x2(bf_lo(rw[e]) + rbf(__uint_as_float(v[2 * j])), bf_hi(rw[e]) + rbf(__uint_as_float(v[2 * j + 1])));
-                        }
-                    }
-                }
-            } else {
-#pragma unroll
-                for (int j = 0; j < 16; ++j) out[j] = pack_bf16x2(__uint_as_float(v[2 * j]), __uint_as_float(v[2 * j + 1]));
-            }
-            if (row < M) {
-                uint4* cp = reinterpret_cast<uint4*>(C + (size_t)row * ldc + n0 + c0);
-#pragma unroll
-                for (int q = 0; q < 4; ++q) cp[q] = make_uint4(out[4 * q], out[4 * q + 1], out[4 * q + 2], out[4 * q + 3]);
-            }
-        }
-        }
-        tc_fence_before();
-    }
-    __syncthreads();
-    if (*aborted) {
-        // After an expired wait (anybody's: the flag is read behind the barrier): copies that were requested still
-        // land in this CTA's shared memory, so the producer waits for the last one of every stage before the CTA exits.
-        if (tid == 0)
-            for (int s = 0; s < Cfg::STAGES && s < issued; ++s) {
-                const int last = ((issued - 1 - s) / Cfg::STAGES) * Cfg::STAGES + s;      // last requested k-block of stage s
-                if (last != drop_kb) mbar_wait_drain(&full[s], (uint32_t)(last / Cfg::STAGES) & 1u);
-            }
-        __syncthreads();
-    }
-    if (warp == 1) tmem_dealloc(tmem_base, Cfg::TMEM_COLS);
-}
 
 // ---------------------------------------------------------------- skinny GEMM for M <= 64 (batched decode)
 // With a handful of activation rows the linears are weight-streaming problems: a
@@ -726,15 +360,6 @@ struct PackedTiles {          // all null / zero for a single prompt
 };
 constexpr size_t FA_SMEM = (size_t)(FA_BQ * FA_LD + FA_NG * 2 * 2 * FA_TILE_ELEMS) * 2;
 
-__device__ __forceinline__ float fast_exp2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ __forceinline__ void cp_async16_zfill(void* smem_dst, const void* gsrc, bool valid) {
-    const uint32_t n = valid ? 16u : 0u;   // 0 source bytes: the 16 destination bytes are zero-filled
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem_dst)), "l"(gsrc), "r"(n) : "memory");
-}
 __device__ __forceinline__ void group_barrier(int group) {
     asm volatile("bar.sync %0, 128;" ::"r"(group + 1) : "memory");
 }
@@ -942,363 +567,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) k_pf_attention(const bf16* __re
     }
 }
 
-// ---------------------------------------------------------------- causal attention on tcgen05 (one prompt)
-// One CTA per (query head, 128-query tile); key tiles of 128 positions.  Both contractions run
-// on the 5th-generation tensor cores with their accumulators in tensor memory:
-//     S = Q K^T     A = Q tile [128 q x 128 d], B = K tile [128 keys x 128 d] straight from the KV cache
-//     O_j = P V     A = P tile [128 q x 128 keys] (bf16) IN TENSOR MEMORY: the softmax warps write the probabilities
-//                   over the scores they came from (tcgen05.st; 64 packed columns of S's 128), so the product
-//                   reads only V from shared memory and nothing crosses the generic / async proxy boundary,
-//                   B = V tile [128 keys x 128 d] straight from the KV cache, read as an MN-major operand
-//                   (the cache rows are contiguous along d, the product contracts over the keys)
-// (128-byte swizzle, fetched by TMA; the V map ends at the last key of the prompt, so the rows of the
-// last tile beyond it arrive as zeros whatever the cache holds there).  Warp 0 feeds the K / V
-// rings, warp 1 issues the MMAs, warps 2-9 hold HALF A QUERY ROW PER THREAD: they read the row's
-// scores from tensor memory (tcgen05.ld), keep the running max / sum and write the probabilities
-// rounded to bf16 as the next MMA's A operand; the output accumulates in tensor memory and is
-// rescaled (tcgen05.ld / st) only when the maximum has grown by more than 2^8.  S is
-// double-buffered: QK^T of tile j + 1 runs while tile j is in the softmax.  Replaces the reference's serial-per-warp kernel and its experimental tiles
-// (csrc/megakernel/fused_prefill_kernels.inl:265-342, 347-445, 486-613).
-constexpr int TA_BQ = 128, TA_BK = 128;
-constexpr int TA_THREADS = 320;                             // warp 0 TMA, warp 1 MMA, warps 2-9 softmax
-constexpr int TA_TILE_BYTES = 128 * 128 * 2;               // two 64-column halves of [128 rows x 128 bytes]
-constexpr int TA_HALF_BYTES = TA_TILE_BYTES / 2;
-constexpr size_t TA_SMEM = (size_t)5 * TA_TILE_BYTES + 1024 /*align*/ + 256 /*barriers*/ + TA_BQ * 8 /*row exchange*/;   // Q, 2 K, 2 V
-static_assert(TA_SMEM <= 232448, "shared memory of one CTA");
-constexpr uint32_t TA_TMEM_COLS = 512;                      // S0 | S1 | O (128 columns each)
-
-
-__global__ void __launch_bounds__(TA_THREADS, 1)
-k_pf_attention_tc(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
-                  bf16* __restrict__ out, int S, int pos0, int layer, int max_seq, unsigned int* status) {
-    pdl_trigger();
-    pdl_wait();
-    extern __shared__ uint8_t ta_raw[];
-    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(ta_raw) + 1023) & ~(uintptr_t)1023);
-    uint8_t* sQ = smem;
-    uint8_t* sK = sQ + TA_TILE_BYTES;            // [2]
-    uint8_t* sV = sK + 2 * TA_TILE_BYTES;        // [2]
-    uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * TA_TILE_BYTES);
-    uint64_t* q_full = bars;                     // 1
-    uint64_t* k_full = bars + 1;                 // 2
-    uint64_t* k_empty = bars + 3;                // 2
-    uint64_t* v_full = bars + 5;                 // 2
-    uint64_t* v_empty = bars + 7;                // 2
-    uint64_t* s_full = bars + 9;                 // 2
-    uint64_t* s_free = bars + 11;                // 2 (256 arrivals)
-    uint64_t* p_full = bars + 13;                // 2 (256 arrivals)
-    uint64_t* o_full = bars + 17;                // 1
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 18);
-    float (*xm)[2] = reinterpret_cast<float(*)[2]>(bars + 20);   // [128][2]: the two half-row maxima (at the end: sums) of a query row
-
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int head = blockIdx.x, g = head / (NQ / NKV);
-    const int q0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * TA_BQ;        // longest query tiles first
-    const int kv_end = min(pos0 + S, pos0 + q0 + TA_BQ);                  // keys any row of the tile may see
-    const int nt = (kv_end + TA_BK - 1) / TA_BK;
-
-    if (tid == 0) {
-        mbar_init(q_full, 1);
-        for (int i = 0; i < 2; ++i) {
-            mbar_init(&k_full[i], 1); mbar_init(&k_empty[i], 1); mbar_init(&v_full[i], 1); mbar_init(&v_empty[i], 1);
-            mbar_init(&s_full[i], 1); mbar_init(&s_free[i], 256); mbar_init(&p_full[i], 256);
-        }
-        mbar_init(o_full, 1);
-        mbar_fence_init();
-    }
-    if (warp == 1) tmem_alloc(tmem_slot, TA_TMEM_COLS);
-    tc_fence_before();
-    __syncthreads();
-    tc_fence_after();
-    const uint32_t tmem_base = *reinterpret_cast<volatile uint32_t*>(tmem_slot);
-    const uint32_t tmem_o = tmem_base + 256;
-
-    if (warp == 0) {
-        if (lane == 0) {
-            mbar_expect_tx(q_full, TA_TILE_BYTES);
-            tma_load_2d(sQ, &tmQ, head * D, q0, q_full);
-            tma_load_2d(sQ + TA_HALF_BYTES, &tmQ, head * D + 64, q0, q_full);
-            const int krow0 = (layer * NKV + g) * max_seq;
-            for (int j = 0; j < nt; ++j) {
-                const int st = j & 1;
-                if (j >= 2 && !mbar_wait(&k_empty[st], (uint32_t)((j >> 1) - 1) & 1u, status)) break;
-                mbar_expect_tx(&k_full[st], TA_TILE_BYTES);
-                tma_load_2d(sK + st * TA_TILE_BYTES, &tmK, 0, krow0 + j * TA_BK, &k_full[st]);
-                tma_load_2d(sK + st * TA_TILE_BYTES + TA_HALF_BYTES, &tmK, 64, krow0 + j * TA_BK, &k_full[st]);
-                if (j >= 2 && !mbar_wait(&v_empty[st], (uint32_t)((j >> 1) - 1) & 1u, status)) break;
-                mbar_expect_tx(&v_full[st], TA_TILE_BYTES);
-                tma_load_3d(sV + st * TA_TILE_BYTES, &tmV, 0, j * TA_BK, layer * NKV + g, &v_full[st]);
-                tma_load_3d(sV + st * TA_TILE_BYTES + TA_HALF_BYTES, &tmV, 64, j * TA_BK, layer * NKV + g, &v_full[st]);
-            }
-        }
-        __syncwarp();
-    } else if (warp == 1) {
-        if (lane == 0) {
-            // instruction descriptor: D = f32, A = B = bf16, both K-major, N = 128, M = 128
-            const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(128 >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
-            const uint32_t idesc_pv = idesc | (1u << 16);    // B (the V tile) is MN-major
-            bool ok = mbar_wait(q_full, 0, status);
-            auto issue_s = [&](int j) {      // S[j & 1] = Q K_j^T
-                const int st = j & 1;
-                ok = ok && mbar_wait(&k_full[st], (uint32_t)(j >> 1) & 1u, status);
-                if (j >= 2) ok = ok && mbar_wait(&s_free[st], (uint32_t)((j >> 1) - 1) & 1u, status);
-                tc_fence_after();
-                if (ok) {
-#pragma unroll
-                    for (int kk = 0; kk < 8; ++kk) {
-                        const uint64_t da = smem_desc_sw128(sQ + (kk >> 2) * TA_HALF_BYTES) + 2 * (kk & 3);
-                        const uint64_t db = smem_desc_sw128(sK + st * TA_TILE_BYTES + (kk >> 2) * TA_HALF_BYTES) + 2 * (kk & 3);
-                        umma_bf16(tmem_base + st * 128, da, db, idesc, kk > 0 ? 1u : 0u);
-                    }
-                }
-                umma_commit(&k_empty[st]);
-                umma_commit(&s_full[st]);
-            };
-            issue_s(0);
-            for (int j = 0; j < nt; ++j) {
-                const int st = j & 1;
-                if (j + 1 < nt) issue_s(j + 1);
-                ok = ok && mbar_wait(&p_full[st], (uint32_t)(j >> 1) & 1u, status);
-                ok = ok && mbar_wait(&v_full[st], (uint32_t)(j >> 1) & 1u, status);
-                tc_fence_after();
-                if (ok) {
-#pragma unroll
-                    for (int kk = 0; kk < 8; ++kk) {
-                        // A = the probabilities, written by the softmax threads over the scores they came from: 16 keys
-                        // of a row are eight 32-bit columns.  B: 16 keys per step = two 1024-byte groups of the
-                        // [keys][64 d] panels (d 0-63 | d 64-127)
-                        const uint64_t db = smem_desc_mn_sw128(sV + st * TA_TILE_BYTES, TA_HALF_BYTES) + (uint64_t)(kk * (2048 >> 4));
-                        umma_bf16_ts(tmem_o, tmem_base + st * 128 + kk * 8, db, idesc_pv, (j > 0 || kk > 0) ? 1u : 0u);   // O accumulates over all key tiles
-                    }
-                }
-                umma_commit(&v_empty[st]);
-                umma_commit(o_full);
-            }
-        }
-        __syncwarp();
-    } else {
-        // softmax warps: TWO threads per query row r = TMEM lane r (warps w and w + 4 share a quarter of the
-        // lanes); thread `half` owns keys [64 half, 64 half + 64) of every key tile and output columns
-        // [64 half, +64).  The two exchange their half-row maxima through shared memory (one 64-thread
-        // named barrier per tile), so both scale by the same running maximum.  The output accumulates in
-        // tensor memory over all key tiles; it is only rescaled when the running maximum has grown by
-        // more than 2^8 since the value the accumulator is scaled to (then p <= 256 in between, exact in
-        // fp32 and harmless in bf16), which after the first tiles practically never happens.  With one
-        // thread per row the 128 exponentials per tile on four warps (one per scheduler) bounded the kernel.
-        const int quarter = warp & 3, half = (warp - 2) >> 2;
-        const int r = quarter * 32 + lane;
-        const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
-        const uint32_t col_off = (uint32_t)(half * 64);
-        const int qpos = pos0 + q0 + r;                       // absolute position of this thread's query
-        const float c = 0.08838834764831845f * 1.4426950408889634f;   // 1/sqrt(128) * log2(e)
-        float m = -INFINITY, l = 0.f;                         // m: the maximum the sums are scaled to (raw score units)
-        bool ok = true;
-        auto pair_sync = [&]() { asm volatile("bar.sync %0, 64;" ::"r"(1 + quarter) : "memory"); };
-        for (int j = 0; j < nt; ++j) {
-            const int st = j & 1;
-            const uint32_t ts = tmem_base + st * 128 + lane_off + col_off;
-            ok = ok && mbar_wait(&s_full[st], (uint32_t)(j >> 1) & 1u, status);
-            tc_fence_after();
-            const int k0 = j * TA_BK + half * 64;             // first key of this thread's half
-            const bool diag = k0 + 63 > qpos;                 // some keys of this half lie beyond the query
-            uint32_t sv[64];
-#pragma unroll
-            for (int cb = 0; cb < 2; ++cb) tmem_ld32_nowait(ts + cb * 32, *reinterpret_cast<uint32_t(*)[32]>(&sv[cb * 32]));
-            tmem_ld_wait();
-            tc_fence_before();
-            mbar_arrive(&s_free[st]);                         // the scores are in registers: S[st] may be overwritten
-            float mh = -INFINITY;
-            if (__any_sync(0xffffffffu, diag)) {              // only the last one or two key tiles of a query tile
-#pragma unroll
-                for (int i = 0; i < 64; ++i) {
-                    if (k0 + i > qpos) sv[i] = 0xff800000u;   // -inf
-                    mh = fmaxf(mh, __uint_as_float(sv[i]));
-                }
-            } else {
-                float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-#pragma unroll
-                for (int i = 0; i < 64; ++i) m4[i & 3] = fmaxf(m4[i & 3], __uint_as_float(sv[i]));
-                mh = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
-            }
-            xm[r][half] = mh;
-            pair_sync();
-            const float mx = fmaxf(xm[r][0], xm[r][1]);       // the same value in both threads of the row
-            pair_sync();                                      // both have read it: the slot is free for the next tile
-            // tcgen05.ld / st are warp-wide: the warp rescales together, rows that need none by 1
-            const bool grow = (mx - m) * c > 8.0f;            // also true for the first tile (m = -inf)
-            // o_full completes once per key tile and is waited on by parity, so every thread consumes EVERY
-            // phase, in order (a parity wait that is two phases behind returns at once): phase j - 1 here if
-            // the accumulator is rescaled, else just before this tile's probabilities are handed over.
-            bool seen_prev = j == 0;
-            if (__any_sync(0xffffffffu, grow)) {
-                const float alpha = grow ? fast_exp2((m - mx) * c) : 1.0f;   // 0 for the first tile
-                if (j > 0) {
-                    // the previous P V product must have landed before the accumulator is touched
-                    ok = ok && mbar_wait(o_full, (uint32_t)(j - 1) & 1u, status);
-                    seen_prev = true;
-                    tc_fence_after();
-#pragma unroll
-                    for (int cb = 0; cb < 2; ++cb) {
-                        uint32_t v[32];
-                        tmem_ld32(tmem_o + lane_off + col_off + cb * 32, v);
-#pragma unroll
-                        for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * alpha);
-                        tmem_st32(tmem_o + lane_off + col_off + cb * 32, v);
-                    }
-                    tc_fence_before();
-                }
-                l *= alpha;
-                if (grow) m = mx;
-            }
-            const float mc = m * c;
-            // (S[st] last held the probabilities of tile j - 2; their product was issued before the Q K^T of this tile)
-            // probabilities -> bf16 pairs -> A operand of the P V product in tensor memory; this thread's 64 keys
-            // are 32 packed columns
-            float rs = 0.f;
-            uint32_t pk[32];
-#pragma unroll
-            for (int i = 0; i < 32; ++i) {
-                const float p0 = fast_exp2(fmaf(__uint_as_float(sv[2 * i]), c, -mc));
-                const float p1 = fast_exp2(fmaf(__uint_as_float(sv[2 * i + 1]), c, -mc));
-                rs += p0 + p1;
-                pk[i] = pack_bf16x2(p0, p1);
-            }
-            // into the columns the scores of keys 0-63 came from (both threads of the row have read theirs: the
-            // exchange above lies in between); 64 keys of the row are 32 columns
-            tmem_st32(tmem_base + st * 128 + lane_off + half * 32, pk);
-            l += rs;
-            if (!seen_prev) ok = ok && mbar_wait(o_full, (uint32_t)(j - 1) & 1u, status);   // P V of tile j - 1 (precedes this tile's anyway)
-            tc_fence_before();
-            mbar_arrive(&p_full[st]);
-        }
-        // the last P V product, then out = O / l (l = the sum of the two half-row sums)
-        ok = ok && mbar_wait(o_full, (uint32_t)(nt - 1) & 1u, status);
-        tc_fence_after();
-        xm[r][half] = l;
-        pair_sync();
-        const float inv = 1.0f / (xm[r][0] + xm[r][1]);
-        bf16* orow = out + (size_t)(q0 + r) * QSZ + head * D + half * 64;
-#pragma unroll
-        for (int cb = 0; cb < 2; ++cb) {
-            uint32_t v[32];
-            tmem_ld32(tmem_o + lane_off + col_off + cb * 32, v);
-            if (q0 + r < S) {
-#pragma unroll
-                for (int q = 0; q < 4; ++q)
-                    reinterpret_cast<uint4*>(orow + cb * 32)[q] =
-                        make_uint4(pack_bf16x2(__uint_as_float(v[8 * q]) * inv, __uint_as_float(v[8 * q + 1]) * inv),
-                                   pack_bf16x2(__uint_as_float(v[8 * q + 2]) * inv, __uint_as_float(v[8 * q + 3]) * inv),
-                                   pack_bf16x2(__uint_as_float(v[8 * q + 4]) * inv, __uint_as_float(v[8 * q + 5]) * inv),
-                                   pack_bf16x2(__uint_as_float(v[8 * q + 6]) * inv, __uint_as_float(v[8 * q + 7]) * inv));
-            }
-        }
-        tc_fence_before();
-    }
-    __syncthreads();
-    if (warp == 1) tmem_dealloc(tmem_base, TA_TMEM_COLS);
-}
-
 // ---------------------------------------------------------------- host side
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-struct MapKey {
-    const void* ptr; uint64_t rows, cols, ld; uint32_t box_rows;
-    uint64_t planes, plane_ld;           // 0, 0 for a matrix
-    bool operator==(const MapKey& o) const {
-        return ptr == o.ptr && rows == o.rows && cols == o.cols && ld == o.ld && box_rows == o.box_rows && planes == o.planes && plane_ld == o.plane_ld;
-    }
-};
-struct MapKeyHash {
-    size_t operator()(const MapKey& k) const {
-        size_t h = reinterpret_cast<size_t>(k.ptr);
-        h ^= k.rows * 0x9e3779b97f4a7c15ull + (h << 6) + (h >> 2);
-        h ^= k.cols * 0xc2b2ae3d27d4eb4full + (h << 6) + (h >> 2);
-        h ^= (k.ld * 31 + k.box_rows) + (h << 6) + (h >> 2);
-        h ^= (k.planes * 0x9e3779b97f4a7c15ull + k.plane_ld) + (h << 6) + (h >> 2);
-        return h;
-    }
-};
-static std::mutex g_map_mu;
-static std::unordered_map<MapKey, CUtensorMap, MapKeyHash> g_maps;
-static EncodeTiledFn g_encode = nullptr;
-
-// Tensor map of a row-major bf16 matrix [rows, cols] with leading dimension ld
-// (elements); box = 64 columns x box_rows rows, 128-byte swizzle, zero fill
-// outside the matrix.  Maps are cached: weight matrices never move.
-// planes > 0: a stack of `planes` such matrices, plane_ld elements apart (a third coordinate selects the plane,
-// and rows beyond `rows` of a plane are filled with zeros instead of running into the next plane).
-static int get_map(const void* ptr, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows, CUtensorMap* out, uint64_t planes = 0,
-                   uint64_t plane_ld = 0) {
-    std::lock_guard<std::mutex> lk(g_map_mu);
-    if (!g_encode) {
-        void* fn = nullptr;
-        cudaDriverEntryPointQueryResult qres;
-        cudaError_t e = cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &qres);
-        if (e != cudaSuccess) return (int)e;
-        if (!fn || qres != cudaDriverEntryPointSuccess) return MQ_ERR_UNSUPPORTED;
-        g_encode = reinterpret_cast<EncodeTiledFn>(fn);
-    }
-    const MapKey key{ptr, rows, cols, ld, box_rows, planes, plane_ld};
-    auto it = g_maps.find(key);
-    if (it != g_maps.end()) { *out = it->second; return MQ_OK; }
-    if (g_maps.size() > 4096) g_maps.clear();
-    const cuuint64_t dims[3] = {cols, rows, planes};
-    const cuuint64_t strides[2] = {ld * 2, plane_ld * 2};
-    const cuuint32_t box[3] = {GM_BK, box_rows, 1};
-    const cuuint32_t estr[3] = {1, 1, 1};
-    CUtensorMap m;
-    const CUresult r = g_encode(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, planes > 0 ? 3 : 2, const_cast<void*>(ptr), dims, strides, box, estr,
-                                CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-                                CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    if (r != CUDA_SUCCESS) return MQ_ERR_BAD_ARG;
-    g_maps.emplace(key, m);
-    *out = m;
-    return MQ_OK;
-}
-
-template <int BN, int EPI, int MT = 1>
-static int launch_gemm(const bf16* A, int lda, const bf16* B, const bf16* B2, bf16* C, const bf16* R, int M, int N, int K, int ldc,
-                       unsigned int* status, cudaStream_t stream, const bf16* B3 = nullptr, int rows0 = 0, int rows1 = 0, int ksplit = 1,
-                       int drop_kb = -1, bool early_b = true) {
-    // early_b: B (B2, B3) are weights, never written by work on this stream; false for caller-supplied operands
-    // rows0 > 0: B, B2, B3 hold rows0, rows1 and N - rows0 - rows1 output columns (concatenated along N)
-    using Cfg = GemmCfg<BN, EPI, MT>;
-    static bool attr_set[64] = {false};
-    int dev = 0;
-    cudaGetDevice(&dev);
-    if (dev >= 0 && dev < 64 && !attr_set[dev]) {
-        cudaError_t e = cudaFuncSetAttribute(k_gemm<BN, EPI, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM);
-        if (e != cudaSuccess) return (int)e;
-        attr_set[dev] = true;
-    }
-    if (N % BN != 0 || K % GM_BK != 0) return MQ_ERR_BAD_ARG;
-    CUtensorMap ma, mb, mb2;
-    int rc = get_map(A, (uint64_t)M, (uint64_t)K, (uint64_t)lda, GM_BM, &ma);
-    if (rc != MQ_OK) return rc;
-    const bool concat = rows0 > 0;
-    if (concat && (rows0 % BN || rows1 % BN || EPI == EPI_SWIGLU)) return MQ_ERR_BAD_ARG;
-    rc = get_map(B, (uint64_t)(concat ? rows0 : N), (uint64_t)K, (uint64_t)K, BN, &mb);
-    if (rc != MQ_OK) return rc;
-    mb2 = mb;
-    CUtensorMap mb3 = mb;
-    if (EPI == EPI_SWIGLU) {
-        rc = get_map(B2, (uint64_t)N, (uint64_t)K, (uint64_t)K, BN, &mb2);
-        if (rc != MQ_OK) return rc;
-    } else if (concat) {
-        rc = get_map(B2, (uint64_t)rows1, (uint64_t)K, (uint64_t)K, BN, &mb2);
-        if (rc != MQ_OK) return rc;
-        rc = get_map(B3, (uint64_t)(N - rows0 - rows1), (uint64_t)K, (uint64_t)K, BN, &mb3);
-        if (rc != MQ_OK) return rc;
-    }
-    if (ksplit < 1 || (ksplit > 1 && EPI != EPI_PARTIAL) || K / GM_BK < ksplit) return MQ_ERR_BAD_ARG;
-    dim3 grid(N / BN, (M + GM_BM * MT - 1) / (GM_BM * MT), ksplit);
-    launch_pdl(k_gemm<BN, EPI, MT>, dim3(grid), dim3(GM_TILE_THREADS), Cfg::SMEM, stream, ma, mb, mb2, mb3, concat ? rows0 / BN : (1 << 30), concat ? rows1 / BN : 0,
-                                                             C, R, M, N, K, ldc, status, drop_kb, early_b ? 1 : 0);
-    return (int)cudaGetLastError();
-}
-
 // Skinny path: part[ks][M][ldp] = X[M,K] * [W0;W1;W2][.,K]^T, K split in `ksplit` slices.
 template <int MPAD>
 static int launch_skinny_t(const bf16* const* W, const int* rowsW, int nW, const bf16* X, int ldx, float* part, int M, int K, int ksplit,
@@ -1879,14 +1148,10 @@ static int prefill_impl(const MqModel* model, const MqDecodeBuffers* dbuf, const
     const bool use_tc = S >= TA_BQ;
     CUtensorMap map_q, map_k, map_v;
     if (use_tc) {
-        static bool ta_attr[64] = {false};
-        if (dev >= 0 && dev < 64 && !ta_attr[dev]) {
-            cudaError_t e = cudaFuncSetAttribute(k_pf_attention_tc, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TA_SMEM);
-            if (e != cudaSuccess) return (int)e;
-            ta_attr[dev] = true;
-        }
-        int mrc = get_map(qkv, (uint64_t)S, (uint64_t)QKV, (uint64_t)QKV, TA_BQ, &map_q);
-        if (mrc == MQ_OK) mrc = get_map(dbuf->k_cache, (uint64_t)model->num_layers * NKV * model->max_seq_len, (uint64_t)D, (uint64_t)D, TA_BK, &map_k);
+        int mrc = get_map(qkv, (uint64_t)S, (uint64_t)D, (uint64_t)QKV, TA_BQ, &map_q, (uint64_t)NQ, (uint64_t)D);
+        if (mrc == MQ_OK)
+            mrc = get_map(dbuf->k_cache, (uint64_t)(pos0 + S), (uint64_t)D, (uint64_t)D, TA_BK, &map_k, (uint64_t)model->num_layers * NKV,
+                          (uint64_t)model->max_seq_len * D);
         if (mrc == MQ_OK)
             mrc = get_map(dbuf->v_cache, (uint64_t)(pos0 + S), (uint64_t)D, (uint64_t)D, TA_BK, &map_v, (uint64_t)model->num_layers * NKV,
                           (uint64_t)model->max_seq_len * D);
@@ -1921,8 +1186,10 @@ static int prefill_impl(const MqModel* model, const MqDecodeBuffers* dbuf, const
                                                          (const bf16*)model->sin_table, (bf16*)dbuf->k_cache, (bf16*)dbuf->v_cache, l, pos0,
                                                          model->max_seq_len, nullptr, 0, nullptr, 0, 0, nullptr);
         if (use_tc) {
-            launch_pdl(k_pf_attention_tc, dim3(NQ, (S + TA_BQ - 1) / TA_BQ), dim3(TA_THREADS), TA_SMEM, stream, map_q, map_k, map_v, attn, S, pos0, l,
-                       model->max_seq_len, status);
+            rc = launch_attention_tc<2, 0, 2>(NQ, map_q, map_k, map_v, map_q, map_k,
+                                              {attn, QSZ, D, S, pos0, NQ / NKV, l * NKV, 8, 0, 0.08838834764831845f * 1.4426950408889634f, nullptr, status},
+                                              stream);
+            if (rc) return rc;
         } else {
             launch_pdl(k_pf_attention, dim3(dim3(NQ, (S + FA_BQ - 1) / FA_BQ)), dim3(FA_THREADS), fa_smem, stream, qkv, (const bf16*)dbuf->k_cache,
                        (const bf16*)dbuf->v_cache, attn, S, pos0, l, model->max_seq_len, PackedTiles());
