@@ -1,4 +1,4 @@
-"""megaqwen_b200 — sm_100a Qwen3-0.6B greedy prefill + decode engine.
+"""megaqwen_b200 — sm_100a greedy prefill + decode engine for Qwen3-0.6B and layer-listed models.
 
 Drop-in for the hot path of the reference's ``megaqwen`` package: the decoder
 object (``MegakernelDecoder`` / ``MegakernelPrefillDecoder``), the generators
@@ -7,7 +7,7 @@ arithmetic runs in hand-written CUDA behind the C ABI of
 ``libmegaqwen_b200.so`` (see include/megaqwen_b200.h).  No Triton, no
 multi-backend dispatch, no CPU fallback.
 """
-from .spec import ModelSpec, QWEN3_0_6B, QWEN3_TINY  # noqa: F401
+from .spec import HybridSpec, ModelSpec, QWEN3_0_6B, QWEN3_TINY  # noqa: F401
 
 
 def __getattr__(name):
@@ -19,6 +19,12 @@ def __getattr__(name):
     if name in ("MegakernelGenerator", "MegakernelPrefillGenerator", "MegakernelFusedPrefillGenerator"):
         from . import generators
         return getattr(generators, name)
+    if name == "HybridDecoder":
+        from .hybrid import HybridDecoder
+        return HybridDecoder
+    if name in ("MODELS", "build_decoder", "find_model"):
+        from . import registry
+        return getattr(registry, name)
     if name == "load_qwen3_weights":
         from .weights import load_qwen3_weights
         return load_qwen3_weights

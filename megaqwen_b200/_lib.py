@@ -1,7 +1,9 @@
-"""ctypes binding of libmegaqwen_b200.so (the C ABI in include/megaqwen_b200.h).
+"""ctypes binding of the package's shared libraries: libmegaqwen_b200.so (the C
+ABI in include/megaqwen_b200.h) and libmegaqwen_hybrid.so
+(include/megaqwen_hybrid.h).
 
-There is no fallback: if the shared library is missing this module raises at
-import time, and the decoder refuses to run without CUDA.
+There is no fallback: loading raises if a library is missing, and the decoders
+refuse to run without CUDA.
 """
 from __future__ import annotations
 
@@ -10,6 +12,8 @@ import os
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.environ.get("MQ_LIB_PATH") or os.path.join(_HERE, "libmegaqwen_b200.so")
+
+HYBRID_LIB_PATH = os.path.join(_HERE, "libmegaqwen_hybrid.so")
 
 MQ_OK = 0
 MQ_ERR = {-1: "bad argument", -2: "sequence too long for the cache or scratch", -3: "unsupported device or geometry",
@@ -106,13 +110,60 @@ SIGNATURES = {
 }
 
 
-def load_library(path: str = LIB_PATH) -> C.CDLL:
+# ---------------------------------------------------------------- include/megaqwen_hybrid.h
+MQH_BF16, MQH_F32 = 0, 1
+MQH_LIGHTNING, MQH_LATENT = 0, 1
+MQH_CHUNK = 128
+MQH_SEGMENT = 32
+
+
+class MqhLayer(C.Structure):
+    _fields_ = [(n, C.c_int) for n in ("kind", "heads", "dim", "vdim", "rank", "rot", "ff", "mix_norm_n")] + [("scale", C.c_float)] + [
+        (n, C.c_void_p) for n in ("norm", "w_in", "w_out", "mix_norm", "decay_pow", "w_ukv", "w_uk_t", "sink", "rope")]
+
+
+class MqhModel(C.Structure):
+    _fields_ = [(n, C.c_int) for n in ("dtype", "width", "norm_n", "vocab", "max_seq")] + [
+        (n, C.c_float) for n in ("embed_scale", "eps", "residual_mult")] + [
+        (n, C.c_int) for n in ("num_layers", "loop_start", "loop_stop", "loop_times")] + [("layers", C.POINTER(MqhLayer))] + [
+        (n, C.c_void_p) for n in ("w_loop", "embed", "final_norm", "head")]
+
+
+class MqhBuffers(C.Structure):
+    _fields_ = [("workspace", C.c_void_p), ("workspace_bytes", C.c_size_t), ("max_tokens", C.c_int), ("run_state", C.POINTER(C.c_void_p)),
+                ("status", C.c_void_p)]
+
+
+_MODEL, _BUF = C.POINTER(MqhModel), C.POINTER(MqhBuffers)
+HYBRID_SIGNATURES = {
+    "mqh_run_count": (C.c_int, [_MODEL]),
+    "mqh_run_layer": (C.c_int, [_MODEL, C.c_int]),
+    "mqh_state_bytes": (C.c_size_t, [_MODEL, C.c_int]),
+    "mqh_state_recurrent": (C.c_int, [_MODEL, C.c_int]),
+    "mqh_in_rows": (C.c_int, [C.POINTER(MqhLayer)]),
+    "mqh_ukv_rows": (C.c_int, [C.POINTER(MqhLayer)]),
+    "mqh_workspace_bytes": (C.c_size_t, [_MODEL, C.c_int]),
+    "mqh_logits_ld": (C.c_int, [_MODEL]),
+    "mqh_decode_launch_count": (C.c_int, [_MODEL]),
+    "mqh_launch_decode": (C.c_int, [_MODEL, _BUF] + [C.c_void_p] * 4 + [C.c_int, C.c_void_p]),
+    "mqh_launch_prefill": (C.c_int, [_MODEL, _BUF, C.c_void_p, C.c_int, C.c_int, C.c_void_p, C.c_int, C.c_void_p, C.c_void_p,
+                                     C.POINTER(C.c_int), C.c_void_p]),
+    "mqh_lightning_scratch_bytes": (C.c_size_t, [C.c_int] * 4),
+    "mqh_launch_lightning": (C.c_int, [C.c_int] + [C.c_void_p] * 6 + [C.c_int] * 5 + [C.c_void_p] * 2),
+    "mqh_launch_causal_attention": (C.c_int, [C.c_int] + [C.c_void_p] * 4 + [C.c_int] + [C.c_void_p] * 3 + [C.c_int] * 6 +
+                                    [C.c_float, C.c_int, C.c_void_p, C.c_void_p]),
+    "mq_launch_fill_iota": SIGNATURES["mq_launch_fill_iota"],
+    "mq_launch_find_first_eos": SIGNATURES["mq_launch_find_first_eos"],
+}
+
+
+def load_library(path: str = LIB_PATH, signatures: dict | None = None) -> C.CDLL:
     if not os.path.exists(path):
         raise ImportError(
             f"{path} is missing: build it with `python -m megaqwen_b200.csrc.build` "
             "(there is no CPU or PyTorch fallback)")
     lib = C.CDLL(path)
-    for name, (res, args) in SIGNATURES.items():
+    for name, (res, args) in (SIGNATURES if signatures is None else signatures).items():
         fn = getattr(lib, name)
         fn.restype = res
         fn.argtypes = args
@@ -120,6 +171,7 @@ def load_library(path: str = LIB_PATH) -> C.CDLL:
 
 
 _lib = None
+_hybrid_lib = None
 
 
 def lib() -> C.CDLL:
@@ -127,6 +179,13 @@ def lib() -> C.CDLL:
     if _lib is None:
         _lib = load_library()
     return _lib
+
+
+def hybrid_lib() -> C.CDLL:
+    global _hybrid_lib
+    if _hybrid_lib is None:
+        _hybrid_lib = load_library(HYBRID_LIB_PATH, HYBRID_SIGNATURES)
+    return _hybrid_lib
 
 
 def check(rc: int, what: str) -> None:

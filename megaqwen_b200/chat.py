@@ -23,8 +23,7 @@ import time
 
 import torch
 
-from .decoder import MegakernelDecoder
-from .weights import load_qwen3_weights
+from .registry import build_decoder
 
 SYSTEM_LINE = "You are a helpful assistant. Be concise and direct. /nothink"
 
@@ -50,15 +49,10 @@ def clean_response(text: str) -> str:
 
 class MegakernelChat:
     def __init__(self, model_name="Qwen/Qwen3-0.6B", max_seq_len=2048, weights=None, device="cuda", out=None):
-        weights = weights or load_qwen3_weights(model_name, max_seq_len=max_seq_len, device=device)
-        self.tokenizer = weights["tokenizer"]
+        self.max_seq_len = int(max_seq_len)
+        self.decoder, self.tokenizer = build_decoder(model_name, self.max_seq_len, weights=weights, device=device)
         if self.tokenizer is None:
             raise RuntimeError("MegakernelChat needs a tokenizer (none was found beside the weights)")
-        self.max_seq_len = int(max_seq_len)
-        self.decoder = MegakernelDecoder(
-            weights["embed_weight"], weights["layer_weights"], weights["final_norm_weight"], weights["lm_head_weight"],
-            weights["cos_table"], weights["sin_table"], len(weights["layer_weights"]) // 11, self.max_seq_len,
-            self.max_seq_len)
         self._out = out or (lambda s: (sys.stdout.write(s), sys.stdout.flush()))
 
     # ------------------------------------------------------------------ generation

@@ -1,0 +1,536 @@
+// Latent attention: every head's keys and values are projections of one normed latent c per
+// token, beside one rotated key part that all heads share; only c and that part are cached.
+//
+// More than one token: keys and values of all cached tokens are expanded once (a product) and
+// the causal attention runs over them, on tcgen05 (tc_attention.cuh) or, for 32-bit models and
+// head shapes that kernel does not hold, in k_causal_rows.
+// One token: the query is carried into the latent space instead (W_uk^T q per head), so that
+// scores and the weighted sum read the cache itself, once for all heads; the sum of latents is
+// carried out again by W_uv.  Three kernels: k_latent_query (that product, rotations, the new
+// cache row), k_latent_attention (splits of the cached tokens), k_latent_merge (sum of the splits
+// with the sink, and W_uv).
+// Scores, weights, rotations and norms are 32-bit; scores are kept in units of log2.
+#include "hy_common.cuh"
+#include "tc_attention.cuh"
+
+namespace mq {
+namespace hy {
+
+constexpr float LOG2E = 1.4426950408889634f;
+
+// The interleaved rotation: elements 2i, 2i + 1 turn by the angle whose cos, sin are rope[i].
+__device__ __forceinline__ float2 rotate_pair(float u, float v, float2 cs) { return make_float2(u * cs.x - v * cs.y, v * cs.x + u * cs.y); }
+__device__ __forceinline__ float2 load2(const float* p) { return __ldcg(reinterpret_cast<const float2*>(p)); }
+__device__ __forceinline__ float2 load2(const bf16* p) {
+    const uint32_t u = ld_cg_u32(p);
+    return make_float2(bf_lo(u), bf_hi(u));
+}
+__device__ __forceinline__ void store2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
+__device__ __forceinline__ void store2(bf16* p, float2 v) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(v.x, v.y); }
+
+// One cache row from the down projection of a token: c = rms(down[0, rank)) * norm, then the rotated key part.
+// NT threads of a CTA.
+template <typename T, int NT>
+__device__ __forceinline__ void write_cache_row(const float* down, const float* norm, int norm_n, float eps, const float* rope_row, T* row, int rank,
+                                                int rot, float* red) {
+    const int tid = threadIdx.x;
+    float ss = 0.f;
+    for (int i = tid * 2; i < rank; i += 2 * NT) {
+        const float2 v = load2(down + i);
+        ss += v.x * v.x + v.y * v.y;
+    }
+    const float inv = 1.0f / sqrtf(cta_sum<NT / 32>(ss, red) / (float)norm_n + eps);
+    for (int i = tid * 2; i < rank; i += 2 * NT) {
+        const float2 v = load2(down + i);
+        store2(row + i, make_float2(v.x * inv * norm[i], v.y * inv * norm[i + 1]));
+    }
+    for (int i = tid; i < rot / 2; i += NT) {
+        const float2 v = load2(down + rank + 2 * i);
+        store2(row + rank + 2 * i, rotate_pair(v.x, v.y, reinterpret_cast<const float2*>(rope_row)[i]));
+    }
+}
+
+// ---------------------------------------------------------------- several tokens
+template <typename T>
+__global__ void __launch_bounds__(128) k_latent_rows(LatentRowsArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float red[4];
+    const int t = blockIdx.x, pos = a.pos0 + t, D = a.rank + a.rot;
+    const float* rope = a.rope + (size_t)pos * a.rot;
+    T* q = reinterpret_cast<T*>(a.q_rot) + (size_t)t * a.heads * a.rot;
+    const int half = a.rot / 2;
+    for (int x = threadIdx.x; x < a.heads * half; x += 128) {
+        const float2 v = load2(q + 2 * x);
+        store2(q + 2 * x, rotate_pair(v.x, v.y, reinterpret_cast<const float2*>(rope)[x % half]));
+    }
+    write_cache_row<T, 128>(a.down + (size_t)t * D, a.norm, a.norm_n, a.eps, rope, reinterpret_cast<T*>(a.cache) + (size_t)pos * D, a.rank, a.rot, red);
+}
+template <typename T>
+int latent_rows(Stream& st, const LatentRowsArgs& a) {
+    return launch(st, k_latent_rows<T>, dim3(a.n), dim3(128), 0, a);
+}
+template int latent_rows<bf16>(Stream&, const LatentRowsArgs&);
+template int latent_rows<float>(Stream&, const LatentRowsArgs&);
+
+// Causal attention without tensor cores: one CTA per (row, head), tiles of 128 keys, online softmax.
+constexpr int CR_KEYS = 128, CR_MAXV = 4;
+template <typename T>
+__global__ void __launch_bounds__(128) k_causal_rows(CausalArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ float cr_q[];                      // [dim + rot]
+    __shared__ float p[CR_KEYS];
+    __shared__ float red[4];
+    const int t = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int nk = a.pos0 + t + 1;
+    const T* q = reinterpret_cast<const T*>(a.q) + ((size_t)t * a.heads + head) * a.dim;
+    const T* qr = reinterpret_cast<const T*>(a.q_rot) + ((size_t)t * a.heads + head) * a.rot;
+    const T* kr = reinterpret_cast<const T*>(a.k_rot);
+    const float c = a.scale * LOG2E;
+    for (int i = tid; i < a.dim; i += 128) cr_q[i] = Elem<T>::get(q[i]);
+    for (int i = tid; i < a.rot; i += 128) cr_q[a.dim + i] = Elem<T>::get(qr[i]);
+    __syncthreads();
+    float m = a.sink ? a.sink[head] * LOG2E : -INFINITY;
+    float l = a.sink ? 1.0f : 0.0f;                      // the sink is a key without a value
+    float acc[CR_MAXV] = {};
+    for (int k0 = 0; k0 < nk; k0 += CR_KEYS) {
+        const int cnt = min(CR_KEYS, nk - k0);
+        float best = -INFINITY;
+        for (int j = warp; j < cnt; j += 4) {
+            const T* k = reinterpret_cast<const T*>(a.k) + ((size_t)(k0 + j) * a.heads + head) * a.dim;
+            float s = 0.f;
+            for (int i = lane * 4; i < a.dim; i += 128) {
+                const float4 kv = load4(k + i), qv = load4(cr_q + i);
+                s = fmaf(kv.x, qv.x, fmaf(kv.y, qv.y, fmaf(kv.z, qv.z, fmaf(kv.w, qv.w, s))));
+            }
+            for (int i = lane; i < a.rot; i += 32) s = fmaf(Elem<T>::get(kr[(size_t)(k0 + j) * a.ld_rot + i]), cr_q[a.dim + i], s);
+            s = warp_sum(s) * c;
+            if (lane == 0) p[j] = s;
+            best = fmaxf(best, s);
+        }
+        if (lane == 0) red[warp] = best;
+        __syncthreads();
+        const float mn = fmaxf(m, fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3])));
+        const float alpha = exp2f(m - mn);
+        if (tid < cnt) p[tid] = exp2f(p[tid] - mn);
+        m = mn;
+        __syncthreads();
+        l = l * alpha + cta_sum<4>(tid < cnt ? p[tid] : 0.f, red);
+#pragma unroll
+        for (int x = 0; x < CR_MAXV; ++x) {
+            const int j = tid + x * 128;
+            if (j >= a.vdim) break;
+            const T* v = reinterpret_cast<const T*>(a.v) + ((size_t)k0 * a.heads + head) * a.vdim + j;
+            float s = 0.f;
+            for (int y = 0; y < cnt; ++y) s = fmaf(p[y], Elem<T>::get(v[(size_t)y * a.heads * a.vdim]), s);
+            acc[x] = acc[x] * alpha + s;
+        }
+        __syncthreads();
+    }
+    T* o = reinterpret_cast<T*>(a.out) + (size_t)t * a.ld_out + (size_t)head * a.vdim;
+#pragma unroll
+    for (int x = 0; x < CR_MAXV; ++x) {
+        const int j = tid + x * 128;
+        if (j < a.vdim) o[j] = Elem<T>::put(acc[x] / l);
+    }
+}
+template <typename T>
+int causal_simt(Stream& st, const CausalArgs& a) {
+    if (a.vdim > CR_MAXV * 128) return MQ_ERR_UNSUPPORTED;
+    return launch(st, k_causal_rows<T>, dim3(a.n, a.heads), dim3(128), (size_t)(a.dim + a.rot) * 4, a);
+}
+template int causal_simt<bf16>(Stream&, const CausalArgs&);
+template int causal_simt<float>(Stream&, const CausalArgs&);
+
+// The tcgen05 kernel holds heads of up to 128 + 64 query / key and 128 value dimensions, and takes a positive scale.
+bool causal_tc_fits(int dim, int rot, int vdim, float scale) { return dim <= 128 && rot <= 64 && vdim <= 128 && scale > 0.f; }
+int causal_tc(Stream& st, const CausalArgs& a) {
+    const uint64_t n = a.n, keys = a.pos0 + a.n, H = a.heads;
+    CUtensorMap mq_, mk, mv, mqr, mkr;
+    int rc = get_map(a.q, n, a.dim, H * a.dim, TA_BQ, &mq_, H, a.dim);
+    if (!rc) rc = get_map(a.q_rot, n, a.rot, H * a.rot, TA_BQ, &mqr, H, a.rot);
+    if (!rc) rc = get_map(a.k, keys, a.dim, H * a.dim, TA_BK, &mk, H, a.dim);
+    if (!rc) rc = get_map(a.k_rot, keys, a.rot, a.ld_rot, TA_BK, &mkr, 1, keys * a.ld_rot);
+    if (!rc) rc = get_map(a.v, keys, a.vdim, H * a.vdim, TA_BK, &mv, H, a.vdim);
+    if (rc) return rc;
+    const AttnTcArgs t = {(bf16*)a.out, a.ld_out, a.vdim, a.n, a.pos0, 1, 0, a.dim / 16, a.rot / 16, a.scale * LOG2E, a.sink, a.status};
+    ++st.launches;
+    const int qp = (a.dim + 63) / 64, vp = (a.vdim + 63) / 64;
+    if (qp == 1 && vp == 1) return launch_attention_tc<1, 1, 1>(a.heads, mq_, mk, mv, mqr, mkr, t, st.s);
+    if (qp == 1 && vp == 2) return launch_attention_tc<1, 1, 2>(a.heads, mq_, mk, mv, mqr, mkr, t, st.s);
+    if (qp == 2 && vp == 1) return launch_attention_tc<2, 1, 1>(a.heads, mq_, mk, mv, mqr, mkr, t, st.s);
+    if (qp == 2 && vp == 2) return launch_attention_tc<2, 1, 2>(a.heads, mq_, mk, mv, mqr, mkr, t, st.s);
+    return MQ_ERR_UNSUPPORTED;
+}
+
+// ---------------------------------------------------------------- one token: query
+// CTA (x, h): q of head h times rows [64 x, 64 x + 64) of its W_uk^T -> qcat[h][..rank).  The extra CTA in x rotates
+// all heads' rotated parts into qcat[h][rank..) and (h = 0) writes the new cache row.
+constexpr int LQ_ROWS = 64, LQ_THREADS = 256;
+template <typename T>
+__global__ void __launch_bounds__(LQ_THREADS) k_latent_query(LatentDecodeArgs a) {
+    extern __shared__ float lq_q[];                      // [dim]
+    __shared__ float red[8];
+    constexpr int EPL = Elem<T>::PER16;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, D = a.rank + a.rot;
+    const bool extra = blockIdx.x == gridDim.x - 1;
+    T* qc = reinterpret_cast<T*>(a.qcat) + (size_t)h * D;
+    // a row of W_uk^T holds dim elements: `lanes` lanes of 16 bytes (a power of two, up to 32), 32 / lanes rows per load
+    int lanes = 1;
+    while (lanes < 32 && lanes * EPL < a.dim) lanes <<= 1;
+    const int per = 32 / lanes, sub = lane / lanes, ln = lane % lanes;
+    const int loads = (LQ_ROWS / 8 + per - 1) / per;     // of this warp's eight rows
+    const T* W = reinterpret_cast<const T*>(a.w_uk_t) + (size_t)h * a.rank * a.dim;
+    const int rbase = blockIdx.x * LQ_ROWS + warp * (LQ_ROWS / 8);
+    uint4 w[8];
+    if (!extra) {
+#pragma unroll
+        for (int x = 0; x < 8; ++x) {
+            const int lr = x * per + sub, r = rbase + lr;
+            const bool ok = x < loads && lr < LQ_ROWS / 8 && r < a.rank && ln * EPL < a.dim;
+            w[x] = ok ? *reinterpret_cast<const uint4*>(W + (size_t)r * a.dim + ln * EPL) : make_uint4(0u, 0u, 0u, 0u);
+        }
+    }
+    pdl_trigger();
+    pdl_wait_cta();
+    if (extra) {
+        int pos = *a.position;
+        if (pos < 0 || pos >= a.max_seq) {
+            if (tid == 0) atomicOr(a.status, MQ_STATUS_BAD_POSITION);
+            pos = pos < 0 ? 0 : a.max_seq - 1;
+        }
+        const float* rope = a.rope + (size_t)pos * a.rot;
+        const T* qr = reinterpret_cast<const T*>(a.q_rot) + (size_t)h * a.rot;
+        for (int i = tid; i < a.rot / 2; i += LQ_THREADS) {
+            const float2 v = load2(qr + 2 * i);
+            store2(qc + a.rank + 2 * i, rotate_pair(v.x, v.y, reinterpret_cast<const float2*>(rope)[i]));
+        }
+        if (h == 0) write_cache_row<T, LQ_THREADS>(a.down, a.norm, a.norm_n, a.eps, rope, reinterpret_cast<T*>(a.cache) + (size_t)pos * D, a.rank, a.rot, red);
+        return;
+    }
+    const T* q = reinterpret_cast<const T*>(a.q) + (size_t)h * a.dim;
+    for (int i = tid; i < a.dim; i += LQ_THREADS) lq_q[i] = Elem<T>::get(__ldcg(q + i));
+    __syncthreads();
+#pragma unroll
+    for (int x = 0; x < 8; ++x) {
+        if (x >= loads) break;
+        const int lr = x * per + sub, r = rbase + lr;
+        const bool ok = lr < LQ_ROWS / 8 && r < a.rank;
+        float s = 0.f;
+        for (int c0 = ln * EPL; c0 < a.dim && ok; c0 += 32 * EPL) {     // one pass unless dim > 32 * EPL
+            const uint4 u = c0 == ln * EPL ? w[x] : *reinterpret_cast<const uint4*>(W + (size_t)r * a.dim + c0);
+            if constexpr (EPL == 8) {
+                const float4 v0 = load4(lq_q + c0), v1 = load4(lq_q + c0 + 4);
+                s = fmaf(bf_lo(u.x), v0.x, s); s = fmaf(bf_hi(u.x), v0.y, s); s = fmaf(bf_lo(u.y), v0.z, s); s = fmaf(bf_hi(u.y), v0.w, s);
+                s = fmaf(bf_lo(u.z), v1.x, s); s = fmaf(bf_hi(u.z), v1.y, s); s = fmaf(bf_lo(u.w), v1.z, s); s = fmaf(bf_hi(u.w), v1.w, s);
+            } else {
+                const float4 v0 = load4(lq_q + c0);
+                s = fmaf(__uint_as_float(u.x), v0.x, s); s = fmaf(__uint_as_float(u.y), v0.y, s);
+                s = fmaf(__uint_as_float(u.z), v0.z, s); s = fmaf(__uint_as_float(u.w), v0.w, s);
+            }
+        }
+        for (int o = lanes >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        if (ok && ln == 0) qc[r] = Elem<T>::put(s);
+    }
+}
+
+// ---------------------------------------------------------------- one token: splits
+// The cached tokens [0, ctx) are dealt to up to `splits` CTAs in equal pieces of whole 64-key tiles.
+constexpr int LA_KEYS = 64;
+int latent_splits(int max_seq) {
+    const int n = (max_seq + LA_KEYS - 1) / LA_KEYS;
+    return n < 148 ? n : 148;
+}
+__device__ __forceinline__ int keys_per_split(int ctx, int splits) {
+    const int tiles = (ctx + LA_KEYS - 1) / LA_KEYS;
+    return ((tiles + splits - 1) / splits) * LA_KEYS;
+}
+__device__ __forceinline__ int clamp_pos(int pos, int max_seq) { return pos < 0 ? 0 : pos >= max_seq ? max_seq - 1 : pos; }
+// A split leaves behind, per head, the sum of its weighted latents [rank], their maximum and the sum of weights.
+size_t latent_parts_floats(int heads, int rank, int max_seq) { return (size_t)latent_splits(max_seq) * heads * (rank + 2); }
+
+// bf16, up to 512 latent dimensions: sixteen heads are the M of mma.sync, so every cached row is read once for all of them.
+constexpr int LA_THREADS = 256, LA_MAXT = 8, LA_PLD = LA_KEYS + 8;
+static size_t la_smem(int D) { return (size_t)(LA_KEYS + 16) * (D + 8) * 2; }
+__global__ void __launch_bounds__(LA_THREADS) k_latent_attention(LatentDecodeArgs a) {
+    extern __shared__ __align__(16) uint8_t la_raw[];
+    __shared__ __align__(16) bf16 sp[16 * LA_PLD];
+    __shared__ float smax[8][16], ssum[8][16];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, D = a.rank + a.rot, ld = D + 8, d8 = D / 8;
+    bf16* sk = reinterpret_cast<bf16*>(la_raw);
+    bf16* sq = sk + LA_KEYS * ld;
+    const bf16* cache = reinterpret_cast<const bf16*>(a.cache);
+    const int h0 = blockIdx.y * 16, split = blockIdx.x;
+    const int pos = clamp_pos(*a.position, a.max_seq), ctx = pos + 1;     // the position was set before this step began
+    const int kps = keys_per_split(ctx, gridDim.x), kbeg = split * kps, kend = min(kbeg + kps, ctx);
+    pdl_trigger();
+    if (kbeg >= kend) return;
+    auto fetch = [&](int k0, int lo, int hi) {            // rows lo .. hi - 1 of the tile at k0; those beyond kend as zeros
+        for (int x = lo * d8 + tid; x < hi * d8; x += LA_THREADS) {
+            const int j = x / d8, col = (x % d8) * 8;
+            const bool ok = k0 + j < kend;
+            cp_async16_zfill(sk + j * ld + col, ok ? cache + (size_t)(k0 + j) * D + col : cache, ok);
+        }
+        cp_async_commit();
+    };
+    // cached rows before the wait; the row of this token (written by the kernel before) after it
+    const bool has_new = kend == ctx && kbeg + LA_KEYS >= ctx;
+    const int jn = pos - kbeg;
+    if (has_new) { fetch(kbeg, 0, jn); fetch(kbeg, jn + 1, LA_KEYS); }
+    else fetch(kbeg, 0, LA_KEYS);
+    pdl_wait_cta();
+    if (has_new) fetch(kbeg, jn, jn + 1);
+    for (int x = tid; x < 16 * d8; x += LA_THREADS) {
+        const int r = x / d8, col = (x % d8) * 8;
+        *reinterpret_cast<uint4*>(sq + r * ld + col) = ld_cg_u4(reinterpret_cast<const bf16*>(a.qcat) + (size_t)(h0 + r) * D + col);
+    }
+    const float c = a.scale * LOG2E;
+    const int ntiles = a.rank / 8, tpw = 2 * ((ntiles + 15) / 16), tile0 = warp * tpw;
+    float acc[LA_MAXT][4];
+#pragma unroll
+    for (int i = 0; i < LA_MAXT; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};               // rows lane / 4, lane / 4 + 8
+    const int row = lane >> 2;
+    for (int k0 = kbeg; k0 < kend; k0 += LA_KEYS) {
+        if (k0 > kbeg) fetch(k0, 0, LA_KEYS);
+        cp_async_wait_all();
+        __syncthreads();
+        // scores of this warp's eight keys; two accumulators break the chain of dependent products
+        float s0[4] = {}, s1[4] = {};
+        const uint32_t qa = smem_u32(sq + (lane & 15) * ld + (lane >> 4) * 8);
+        const uint32_t kb = smem_u32(sk + (warp * 8 + row) * ld + (lane & 3) * 2);
+        int ks = 0;
+        for (; ks + 1 < D / 16; ks += 2) {
+            uint32_t q4[4], r4[4];
+            ldsm4(q4, qa + ks * 32);
+            ldsm4(r4, qa + ks * 32 + 32);
+            mma16816(s0, q4, lds32(kb + ks * 32), lds32(kb + ks * 32 + 16));
+            mma16816(s1, r4, lds32(kb + ks * 32 + 32), lds32(kb + ks * 32 + 48));
+        }
+        if (ks < D / 16) {
+            uint32_t q4[4];
+            ldsm4(q4, qa + ks * 32);
+            mma16816(s0, q4, lds32(kb + ks * 32), lds32(kb + ks * 32 + 16));
+        }
+        float s[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int key = k0 + warp * 8 + 2 * (lane & 3) + (e & 1);
+            s[e] = key < kend ? (s0[e] + s1[e]) * c : -INFINITY;
+        }
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            float v = fmaxf(s[2 * h], s[2 * h + 1]);
+            v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 1));
+            v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 2));
+            if ((lane & 3) == 0) smax[warp][row + 8 * h] = v;
+        }
+        __syncthreads();
+        float alpha[2];
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            float mn = m[h];
+#pragma unroll
+            for (int w = 0; w < 8; ++w) mn = fmaxf(mn, smax[w][row + 8 * h]);
+            alpha[h] = exp2f(m[h] - mn);
+            m[h] = mn;
+            const float p0 = exp2f(s[2 * h] - mn), p1 = exp2f(s[2 * h + 1] - mn);
+            *reinterpret_cast<uint32_t*>(sp + (row + 8 * h) * LA_PLD + warp * 8 + 2 * (lane & 3)) = pack_bf16x2(p0, p1);
+            float v = p0 + p1;
+            v += __shfl_xor_sync(0xffffffffu, v, 1);
+            v += __shfl_xor_sync(0xffffffffu, v, 2);
+            if ((lane & 3) == 0) ssum[warp][row + 8 * h] = v;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            float v = 0.f;
+#pragma unroll
+            for (int w = 0; w < 8; ++w) v += ssum[w][row + 8 * h];
+            l[h] = l[h] * alpha[h] + v;
+        }
+#pragma unroll
+        for (int i = 0; i < LA_MAXT; ++i) { acc[i][0] *= alpha[0]; acc[i][1] *= alpha[0]; acc[i][2] *= alpha[1]; acc[i][3] *= alpha[1]; }
+#pragma unroll
+        for (int ks = 0; ks < LA_KEYS / 16; ++ks) {
+            uint32_t p4[4];
+            ldsm4(p4, smem_u32(sp + (lane & 15) * LA_PLD + ks * 16 + (lane >> 4) * 8));
+#pragma unroll
+            for (int i = 0; i < LA_MAXT; i += 2) {
+                if (i >= tpw || tile0 + i >= ntiles) break;
+                uint32_t b[4];
+                ldsm4_t(b, smem_u32(sk + (ks * 16 + (lane & 15)) * ld + (tile0 + i) * 8 + (lane >> 4) * 8));
+                mma16816(acc[i], p4, b[0], b[1]);
+                mma16816(acc[i + 1], p4, b[2], b[3]);
+            }
+        }
+        __syncthreads();                                   // keys, weights and maxima are overwritten by the next tile
+    }
+    const int heads_here = min(16, a.heads - h0);
+    float* part = a.parts + ((size_t)split * a.heads + h0) * (a.rank + 2);
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        const int r = row + 8 * h;
+        if (r >= heads_here) continue;
+        float* dst = part + (size_t)r * (a.rank + 2);
+#pragma unroll
+        for (int i = 0; i < LA_MAXT; ++i) {
+            if (i >= tpw || tile0 + i >= ntiles) break;
+            *reinterpret_cast<float2*>(dst + (tile0 + i) * 8 + 2 * (lane & 3)) = make_float2(acc[i][2 * h], acc[i][2 * h + 1]);
+        }
+        if (warp == 0 && (lane & 3) == 0) *reinterpret_cast<float2*>(dst + a.rank) = make_float2(m[h], l[h]);
+    }
+}
+
+// The same split for 32-bit caches and larger latents: one CTA per (split, head).
+constexpr int LP_THREADS = 128, LP_MAXC = 16;
+template <typename T>
+__global__ void __launch_bounds__(LP_THREADS) k_latent_attention_plain(LatentDecodeArgs a) {
+    extern __shared__ float lp_q[];                        // [rank + rot]
+    __shared__ float p[LA_KEYS];
+    __shared__ float red[4];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, D = a.rank + a.rot, head = blockIdx.y, split = blockIdx.x;
+    const T* cache = reinterpret_cast<const T*>(a.cache);
+    pdl_trigger();
+    pdl_wait_cta();
+    const int pos = clamp_pos(*a.position, a.max_seq), ctx = pos + 1;
+    const int kps = keys_per_split(ctx, gridDim.x), kbeg = split * kps, kend = min(kbeg + kps, ctx);
+    if (kbeg >= kend) return;
+    for (int i = tid; i < D; i += LP_THREADS) lp_q[i] = Elem<T>::get(__ldcg(reinterpret_cast<const T*>(a.qcat) + (size_t)head * D + i));
+    __syncthreads();
+    const float c = a.scale * LOG2E;
+    float m = -INFINITY, l = 0.f, acc[LP_MAXC] = {};
+    for (int k0 = kbeg; k0 < kend; k0 += LA_KEYS) {
+        const int cnt = min(LA_KEYS, kend - k0);
+        float best = -INFINITY;
+        for (int j = warp; j < cnt; j += 4) {
+            float s = 0.f;
+            for (int i = lane * 4; i < D; i += 128) {
+                const float4 kv = load4_cg(cache + (size_t)(k0 + j) * D + i), qv = load4(lp_q + i);
+                s = fmaf(kv.x, qv.x, fmaf(kv.y, qv.y, fmaf(kv.z, qv.z, fmaf(kv.w, qv.w, s))));
+            }
+            s = warp_sum(s) * c;
+            if (lane == 0) p[j] = s;
+            best = fmaxf(best, s);
+        }
+        if (lane == 0) red[warp] = best;
+        __syncthreads();
+        const float mn = fmaxf(m, fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3])));
+        const float alpha = exp2f(m - mn);
+        m = mn;
+        if (tid < cnt) p[tid] = exp2f(p[tid] - mn);
+        __syncthreads();
+        l = l * alpha + cta_sum<4>(tid < cnt ? p[tid] : 0.f, red);
+#pragma unroll
+        for (int x = 0; x < LP_MAXC; ++x) {
+            const int i = tid + x * LP_THREADS;
+            if (i >= a.rank) break;
+            float s = 0.f;
+            for (int j = 0; j < cnt; ++j) s = fmaf(p[j], Elem<T>::get(__ldcg(cache + (size_t)(k0 + j) * D + i)), s);
+            acc[x] = acc[x] * alpha + s;
+        }
+        __syncthreads();
+    }
+    float* dst = a.parts + ((size_t)split * a.heads + head) * (a.rank + 2);
+#pragma unroll
+    for (int x = 0; x < LP_MAXC; ++x) {
+        const int i = tid + x * LP_THREADS;
+        if (i < a.rank) dst[i] = acc[x];
+    }
+    if (tid == 0) { dst[a.rank] = m; dst[a.rank + 1] = l; }
+}
+
+// ---------------------------------------------------------------- one token: merge
+// CTA (x, h): the latent sum of head h over all splits, the sink in the denominator, then rows [32 x, 32 x + 32) of its W_uv.
+constexpr int LM_ROWS = 32, LM_THREADS = 256, LM_PRE = 2;
+template <typename T>
+__global__ void __launch_bounds__(LM_THREADS) k_latent_merge(LatentDecodeArgs a, int splits) {
+    extern __shared__ float lm_c[];                        // [rank], then the weight of every split
+    constexpr int EPL = Elem<T>::PER16;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y;
+    float* ws = lm_c + a.rank;
+    const int r0 = blockIdx.x * LM_ROWS + warp * (LM_ROWS / 8);
+    const T* W = reinterpret_cast<const T*>(a.w_uv) + (size_t)h * a.vdim * a.rank;
+    uint4 w[LM_ROWS / 8][LM_PRE];
+#pragma unroll
+    for (int x = 0; x < LM_ROWS / 8; ++x)
+#pragma unroll
+        for (int s = 0; s < LM_PRE; ++s) {
+            const int c0 = (s * 32 + lane) * EPL;
+            w[x][s] = r0 + x < a.vdim && c0 < a.rank ? *reinterpret_cast<const uint4*>(W + (size_t)(r0 + x) * a.rank + c0) : make_uint4(0u, 0u, 0u, 0u);
+        }
+    pdl_trigger();
+    pdl_wait_cta();
+    const int ctx = clamp_pos(*a.position, a.max_seq) + 1;
+    const int kps = keys_per_split(ctx, splits), active = (ctx + kps - 1) / kps;
+    const float* part = a.parts + (size_t)h * (a.rank + 2);
+    const size_t stride = (size_t)a.heads * (a.rank + 2);
+    for (int s = tid; s < active; s += LM_THREADS) ws[s] = __ldcg(part + s * stride + a.rank);
+    __syncthreads();
+    const float sink = a.sink ? a.sink[h] * LOG2E : -INFINITY;
+    float m = sink;
+    for (int s = 0; s < active; ++s) m = fmaxf(m, ws[s]);
+    __syncthreads();
+    float l = 0.f;
+    for (int s = tid; s < active; s += LM_THREADS) {
+        const float e = exp2f(ws[s] - m);
+        l += e * __ldcg(part + s * stride + a.rank + 1);
+        ws[s] = e;
+    }
+    __shared__ float red[8];
+    const float inv = 1.0f / (cta_sum<8>(l, red) + exp2f(sink - m));
+    for (int i = tid; i < a.rank; i += LM_THREADS) {
+        float s = 0.f;
+#pragma unroll 8
+        for (int x = 0; x < active; ++x) s = fmaf(ws[x], __ldcg(part + x * stride + i), s);
+        lm_c[i] = s * inv;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int x = 0; x < LM_ROWS / 8; ++x) {
+        const int r = r0 + x;
+        if (r >= a.vdim) break;
+        float s = 0.f;
+        int seg = 0;
+        for (int c0 = lane * EPL; c0 < a.rank; c0 += 32 * EPL, ++seg) {
+            const uint4 u = seg == 0 ? w[x][0] : seg == 1 ? w[x][1] : *reinterpret_cast<const uint4*>(W + (size_t)r * a.rank + c0);
+            if constexpr (EPL == 8) {
+                const float4 v0 = load4(lm_c + c0), v1 = load4(lm_c + c0 + 4);
+                s = fmaf(bf_lo(u.x), v0.x, s); s = fmaf(bf_hi(u.x), v0.y, s); s = fmaf(bf_lo(u.y), v0.z, s); s = fmaf(bf_hi(u.y), v0.w, s);
+                s = fmaf(bf_lo(u.z), v1.x, s); s = fmaf(bf_hi(u.z), v1.y, s); s = fmaf(bf_lo(u.w), v1.z, s); s = fmaf(bf_hi(u.w), v1.w, s);
+            } else {
+                const float4 v0 = load4(lm_c + c0);
+                s = fmaf(__uint_as_float(u.x), v0.x, s); s = fmaf(__uint_as_float(u.y), v0.y, s);
+                s = fmaf(__uint_as_float(u.z), v0.z, s); s = fmaf(__uint_as_float(u.w), v0.w, s);
+            }
+        }
+        s = warp_sum(s);
+        if (lane == 0) reinterpret_cast<T*>(a.out)[(size_t)h * a.vdim + r] = Elem<T>::put(s);
+    }
+}
+
+template <typename T> struct IsBf16 { static constexpr bool v = false; };
+template <> struct IsBf16<bf16> { static constexpr bool v = true; };
+template <typename T>
+int latent_decode(Stream& st, const LatentDecodeArgs& a) {
+    const int splits = latent_splits(a.max_seq), D = a.rank + a.rot;
+    int rc = launch(st, k_latent_query<T>, dim3((a.rank + LQ_ROWS - 1) / LQ_ROWS + 1, a.heads), dim3(LQ_THREADS), (size_t)a.dim * 4, a);
+    if (rc) return rc;
+    if (IsBf16<T>::v && a.rank <= LA_MAXT * 64 && la_smem(D) <= 200 * 1024) {
+        rc = allow_smem(k_latent_attention, la_smem(D));
+        if (!rc) rc = launch(st, k_latent_attention, dim3(splits, (a.heads + 15) / 16), dim3(LA_THREADS), la_smem(D), a);
+    } else {
+        if (a.rank > LP_THREADS * LP_MAXC) return MQ_ERR_UNSUPPORTED;
+        rc = launch(st, k_latent_attention_plain<T>, dim3(splits, a.heads), dim3(LP_THREADS), (size_t)D * 4, a);
+    }
+    if (rc) return rc;
+    return launch(st, k_latent_merge<T>, dim3((a.vdim + LM_ROWS - 1) / LM_ROWS, a.heads), dim3(LM_THREADS), (size_t)(a.rank + splits) * 4, a, splits);
+}
+template int latent_decode<bf16>(Stream&, const LatentDecodeArgs&);
+template int latent_decode<float>(Stream&, const LatentDecodeArgs&);
+
+}  // namespace hy
+}  // namespace mq

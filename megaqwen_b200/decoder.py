@@ -15,17 +15,14 @@ import torch
 
 from . import _lib
 from ._lib import MqDecodeBuffers, MqKvFp8, MqLayerWeights, MqModel, MqPrefillBuffers
+from .engine import DecodeEngine, _ptr
 
 _HIDDEN, _INTER, _NQ, _NKV, _D = 1024, 3072, 16, 8, 128
 _LAYER_SHAPES = [(_HIDDEN,), (_NQ * _D, _HIDDEN), (_NKV * _D, _HIDDEN), (_NKV * _D, _HIDDEN), (_D,), (_D,),
                  (_HIDDEN, _NQ * _D), (_HIDDEN,), (_INTER, _HIDDEN), (_INTER, _HIDDEN), (_HIDDEN, _INTER)]
 
 
-def _ptr(t: torch.Tensor) -> int:
-    return t.data_ptr()
-
-
-class MegakernelDecoder:
+class MegakernelDecoder(DecodeEngine):
     """Batch-1 greedy decoder.
 
     ``position()`` is the number of tokens consumed.  ``decode_step(t)`` writes
@@ -48,19 +45,17 @@ class MegakernelDecoder:
                  num_layers, max_seq_len, max_prefill_len=512, *w4_args, kv_fp8=None, **w4_kwargs):
         if not torch.cuda.is_available():
             raise RuntimeError("megaqwen_b200 needs a CUDA device (sm_100a); there is no CPU fallback")
-        self._lib = _lib.lib()
+        lib = _lib.lib()
         for extra in list(w4_args) + list(w4_kwargs.values()):
             if extra is not None and hasattr(extra, "__len__") and len(extra) > 0:
                 raise RuntimeError("W4 / paged-KV options are not supported by this engine")
         if len(layer_weights) != 11 * num_layers:
             raise RuntimeError(f"layer_weights must hold 11 tensors per layer, got {len(layer_weights)} for {num_layers} layers")
-        self.device = embed_weight.device
-        if self.device.type != "cuda":
+        device = embed_weight.device
+        if device.type != "cuda":
             raise RuntimeError("weights must live on a CUDA device")
         self.num_layers_ = int(num_layers)
-        self.max_seq_len_ = int(max_seq_len)
-        self.max_prefill_len_ = int(max_prefill_len)
-        self.vocab_size_ = int(embed_weight.shape[0])
+        self._init_engine(lib, device, int(embed_weight.shape[0]), max_seq_len, max_prefill_len)
 
         def chk(t, shape, name):
             if t.dtype != torch.bfloat16 or not t.is_contiguous() or t.device != self.device or tuple(t.shape) != tuple(shape):
@@ -97,11 +92,6 @@ class MegakernelDecoder:
             self._partials = torch.zeros(self._lib.mq_decode_partials_bytes(self.max_seq_len_) // 4, dtype=torch.float32, device=dev)
             self._counters = torch.zeros(16, dtype=i32, device=dev)
             self._slot = torch.zeros(1, dtype=torch.int64, device=dev)
-            # [0] = output token of single steps, [1] = sticky status word
-            self._scalars = torch.zeros(4, dtype=i32, device=dev)
-            self._in_token = torch.zeros(1, dtype=i32, device=dev)
-            self._pos_dev = torch.zeros(1, dtype=i32, device=dev)
-            self._logits = None
             self._pf = None            # prefill activation buffers, allocated at the first prefill
             self._pf_tensors = None
             self.use_gemm_prefill = True
@@ -114,10 +104,6 @@ class MegakernelDecoder:
             # opt-in: measured on B200 the graph-replayed per-phase kernels are still faster
             # (389 vs 425 us/token at context 1, 477 vs 508 at 2048)
             self.use_persistent = False
-            self._chain_cap = 0
-            self._chain_tokens = None
-            self._chain_pos = None
-            self._graphs = {}
             if kv_fp8 is None:
                 kv_fp8 = os.environ.get("MEGAQWEN_SPLIT_KV_FP8", "0").strip().lower() in ("1", "true", "yes", "on")
             self.kv_fp8 = bool(kv_fp8)
@@ -132,16 +118,11 @@ class MegakernelDecoder:
         self._buf = MqDecodeBuffers(_ptr(self.k_cache_), _ptr(self.v_cache_), _ptr(self._hidden), _ptr(self._qkv),
                                     _ptr(self._attn), _ptr(self._act), _ptr(self._partials), _ptr(self._counters),
                                     _ptr(self._slot), _ptr(self._scalars) + 4, nsplit)
-        self.position_ = 0
-        self.use_pdl = True
-        self.use_step_graph = True  # decode_step replays a captured one-step graph instead of 141 eager launches
-        self._step_graph = None
-        self._step_graph_pdl = None
-        self.launches = 0          # kernels launched through the C ABI by this object
 
     # ------------------------------------------------------------------ helpers
-    def _stream(self) -> int:
-        return torch.cuda.current_stream(self.device).cuda_stream
+    @property
+    def step_launches(self) -> int:
+        return 5 * self.num_layers_ + 1
 
     def _launch(self, in_ptr: int, out_ptr: int, pos_ptr: int, logits_ptr, chained: bool) -> None:
         flags = (_lib.MQ_FLAG_CHAINED if chained else 0) | (0 if self.use_pdl else _lib.MQ_FLAG_NO_PDL)
@@ -152,7 +133,7 @@ class MegakernelDecoder:
             rc = self._lib.mq_launch_decode(C.byref(self._model), C.byref(self._buf), in_ptr, out_ptr, pos_ptr,
                                             logits_ptr, flags, self._stream())
         _lib.check(rc, "mq_launch_decode")
-        self.launches += 5 * self.num_layers_ + 1
+        self.launches += self.step_launches
 
     def _kv8_sync(self) -> None:
         """Before a decode launch: rows written by a prefill since the last decode are quantised into
@@ -165,37 +146,18 @@ class MegakernelDecoder:
             self.launches += 1
             self._kv8_ready = self.position_
 
-    def _check_status(self, status: int) -> None:
-        if status:
-            self._scalars[1] = 0
-            what = []
-            if status & _lib.MQ_STATUS_WAIT_TIMEOUT:
-                what.append("a bounded device-side wait expired")
-            if status & _lib.MQ_STATUS_BAD_POSITION:
-                what.append("position outside the KV cache")
-            if status & _lib.MQ_STATUS_BAD_TOKEN:
-                what.append("token id outside the vocabulary")
-            raise RuntimeError("megaqwen_b200 device status: " + ", ".join(what))
+    _before_decode = _kv8_sync
 
-    def check_status(self) -> None:
-        """Read the sticky device status word (one 4-byte copy) and raise if set."""
-        self._check_status(int(self._scalars[1].item()))
+    def _after_decode(self) -> None:
+        self._kv8_ready = self.position_
 
-    def _ensure_chain(self, n: int) -> None:
-        if n > self._chain_cap:
-            cap = max(n, 64)
-            self._chain_tokens = torch.zeros(cap + 1, dtype=torch.int32, device=self.device)
-            self._chain_pos = torch.zeros(cap, dtype=torch.int32, device=self.device)
-            self._chain_cap = cap
-            self._graphs = {}
+    def _chain_persistent(self, tokens, num_steps: int) -> bool:
+        if not self.use_persistent or self.kv_fp8 or self.position_ + num_steps > self._stream_max_context:
+            return False
+        self._launch_stream(_ptr(tokens), None, _ptr(tokens) + 4, num_steps, None, False, None)
+        return True
 
     # ------------------------------------------------------------------ reference API
-    def position(self) -> int:
-        return self.position_
-
-    def max_prefill_len(self) -> int:
-        return self.max_prefill_len_
-
     def get_k_cache(self) -> torch.Tensor:
         return self.k_cache_
 
@@ -212,113 +174,12 @@ class MegakernelDecoder:
             self.v_cache_fp8_.zero_()
             self.kv_scales_.fill_(1.0)
 
-    def _single(self, input_token_id: int, logits_ptr) -> int:
-        if self.position_ >= self.max_seq_len_:
-            raise RuntimeError("decode_step would exceed max_seq_len")
-        with torch.cuda.device(self.device):
-            # scalar fills carry the value as a kernel argument: no host buffer to race on
-            self._in_token.fill_(int(input_token_id))
-            self._pos_dev.fill_(self.position_)
-            self._kv8_sync()
-            if logits_ptr is None and self.use_step_graph:
-                self._replay_step_graph()
-            else:
-                self._launch(_ptr(self._in_token), _ptr(self._scalars), _ptr(self._pos_dev), logits_ptr, False)
-            self.position_ += 1
-            self._kv8_ready = self.position_
-            tok, status = self._scalars[:2].tolist()
-        self._check_status(status)
-        return tok
-
-    def _replay_step_graph(self) -> None:
-        """One decode step (token and position in device scalars) captured once and replayed:
-        the host cost of a step is one graph launch instead of 141 kernel launches."""
-        if self._step_graph is None or self._step_graph_pdl != self.use_pdl:
-            g = torch.cuda.CUDAGraph()
-            launches0 = self.launches
-            s = torch.cuda.Stream(device=self.device)
-            s.wait_stream(torch.cuda.current_stream(self.device))
-            with torch.cuda.stream(s):
-                with torch.cuda.graph(g, stream=s):
-                    self._launch(_ptr(self._in_token), _ptr(self._scalars), _ptr(self._pos_dev), None, False)
-            torch.cuda.current_stream(self.device).wait_stream(s)
-            self.launches = launches0
-            self._step_graph, self._step_graph_pdl = g, self.use_pdl
-        self._step_graph.replay()
-        self.launches += 5 * self.num_layers_ + 1
-
-    def decode_step(self, input_token_id: int) -> int:
-        return self._single(input_token_id, None)
-
-    def decode_step_logits(self, input_token_id: int):
-        """One step that also returns the bf16-rounded logits as fp32 [vocab]
-        (reference: launch_ldg_decode_with_logits, chat.py:241-314)."""
-        if self._logits is None:
-            self._logits = torch.empty(self.vocab_size_, dtype=torch.float32, device=self.device)
-        tok = self._single(input_token_id, _ptr(self._logits))
-        return tok, self._logits.clone()
-
-    def _chain(self, first_token, num_steps: int, use_graph: bool, what: str = "decode_steps") -> torch.Tensor:
-        """Device-resident chain token[i] -> token[i+1]; returns the view of the
-        num_steps generated tokens (cuda int32).  No host synchronisation."""
-        if num_steps <= 0:
-            return torch.empty(0, dtype=torch.int32, device=self.device)
-        # the reference's bound (bindings_prefill.cpp:1049-1051, 1092): the last cache row stays unused
-        if self.position_ + num_steps >= self.max_seq_len_:
-            raise RuntimeError(f"{what} would exceed max_seq_len")
-        with torch.cuda.device(self.device):
-            self._ensure_chain(num_steps)
-            self._kv8_sync()
-            tk, ps = self._chain_tokens, self._chain_pos
-            if torch.is_tensor(first_token):
-                tk[0:1].copy_(first_token.reshape(1).to(torch.int32), non_blocking=True)
-            else:
-                tk[0:1].fill_(int(first_token))
-            if self.use_persistent and not self.kv_fp8 and use_graph and self.position_ + num_steps <= self._stream_max_context:
-                self._launch_stream(_ptr(tk), None, _ptr(tk) + 4, num_steps, None, False, None)
-                self.position_ += num_steps
-                return tk[1:num_steps + 1]
-            _lib.check(self._lib.mq_launch_fill_iota(_ptr(ps), self.position_, num_steps, self._stream()), "mq_launch_fill_iota")
-            self.launches += 1
-            if use_graph:
-                self._replay_graph(num_steps)
-            else:
-                for i in range(num_steps):
-                    self._launch(_ptr(tk) + 4 * i, _ptr(tk) + 4 * (i + 1), _ptr(ps) + 4 * i, None, i > 0)
-            self.position_ += num_steps
-            self._kv8_ready = self.position_
-            return tk[1:num_steps + 1]
-
-    def _replay_graph(self, num_steps: int) -> None:
-        key = (num_steps, self.use_pdl)      # the PDL attribute is baked into the captured launches
-        g = self._graphs.get(key)
-        tk, ps = self._chain_tokens, self._chain_pos
-        if g is None:
-            g = torch.cuda.CUDAGraph()
-            launches0 = self.launches
-            # capture on a side stream as torch requires; the chain reads tokens[0]
-            # and positions[] which are refreshed before every replay
-            s = torch.cuda.Stream(device=self.device)
-            s.wait_stream(torch.cuda.current_stream(self.device))
-            with torch.cuda.stream(s):
-                with torch.cuda.graph(g, stream=s):
-                    for i in range(num_steps):
-                        self._launch(_ptr(tk) + 4 * i, _ptr(tk) + 4 * (i + 1), _ptr(ps) + 4 * i, None, i > 0)
-            torch.cuda.current_stream(self.device).wait_stream(s)
-            self.launches = launches0
-            self._graphs[key] = g
-        g.replay()
-        self.launches += num_steps * (5 * self.num_layers_ + 1)
-
-    def decode_steps_cuda(self, first_token, num_steps: int) -> torch.Tensor:
-        return self._chain(first_token, num_steps, False).clone()
-
     def decode_steps_cuda_graph(self, first_token, num_steps: int) -> torch.Tensor:
         """Per-phase kernels replayed from a CUDA graph (reference:
         decode_steps_cuda_graph, bindings_prefill.cpp:1082-1150)."""
         keep, self.use_persistent = self.use_persistent, False
         try:
-            return self._chain(first_token, num_steps, True, "decode_steps_cuda_graph").clone()
+            return super().decode_steps_cuda_graph(first_token, num_steps)
         finally:
             self.use_persistent = keep
 
@@ -391,69 +252,6 @@ class MegakernelDecoder:
             self.position_ += 1
         self.check_status()
         return cycles
-
-    def decode_steps(self, first_token_id: int, num_steps: int) -> torch.Tensor:
-        out = self._chain(first_token_id, num_steps, True)
-        host = torch.cat([out, self._scalars[1:2]]).cpu()
-        self._check_status(int(host[-1]))
-        return host[:-1]
-
-    def decode_greedy_cuda(self, first_token, max_new_tokens: int, eos_ids, chunk: int = 32):
-        """Greedy loop with tokens kept on the device; the EOS scan and one 4-byte
-        read happen once per chunk.  Same contract as the reference
-        (bindings_prefill.cpp:1159-1349): the result holds the CONSUMED tokens,
-        i.e. per chunk ``[next_token] + generated[:-1]``, so ``out[0]`` is
-        ``first_token`` and the last token a chunk generated is carried into the
-        next chunk instead of being returned; EOS is searched in
-        ``generated[:-1]`` of each chunk and excluded from the result;
-        ``position()`` advances by whole chunks (the cache rows past an EOS were
-        computed and stay).  Returns (tokens cuda int32[len], len, stop_reason)
-        with stop_reason 0 = max_new_tokens, 1 = EOS."""
-        max_new = int(max_new_tokens)
-        if max_new <= 0:
-            return torch.empty(0, dtype=torch.int32, device=self.device), 0, 0
-        if chunk <= 0:
-            chunk = 32
-        if eos_ids is None or len(eos_ids) == 0:
-            raise RuntimeError("eos_ids must be a non-empty int32 tensor")
-        eos = torch.as_tensor(eos_ids).to(device=self.device, dtype=torch.int32).contiguous()
-        out = torch.empty(max_new, dtype=torch.int32, device=self.device)
-        hit = torch.empty(1, dtype=torch.int32, device=self.device)
-        gen_len, stop_reason, cur = 0, 0, first_token
-        while gen_len < max_new:
-            steps = min(chunk, max_new - gen_len)
-            tail = self._chain(cur, steps, steps == chunk)          # view of tokens[1 .. steps]
-            tokens = self._chain_tokens                             # tokens[0] = consumed token of this chunk
-            out[gen_len:gen_len + steps].copy_(tokens[:steps])
-            stop_pos = -1
-            if steps > 1:
-                hit.fill_(steps - 1)
-                _lib.check(self._lib.mq_launch_find_first_eos(_ptr(tokens) + 4, steps - 1, _ptr(eos), eos.numel(), _ptr(hit),
-                                                              self._stream()), "mq_launch_find_first_eos")
-                self.launches += 1
-                idx = int(hit.item())
-                if idx < steps - 1:
-                    stop_pos = idx + 1          # tokens kept from this chunk; the EOS itself is dropped
-            if stop_pos >= 0:
-                gen_len += stop_pos
-                stop_reason = 1
-                break
-            gen_len += steps
-            cur = tail[steps - 1:steps].clone()
-        self.check_status()
-        return out[:gen_len], gen_len, stop_reason
-
-    def _check_prefill(self, ids: torch.Tensor, pos0: int) -> int:
-        """The reference's checks and texts (bindings_prefill.cpp:731-739); the ASR caller
-        matches on them (megaqwen/qwen3_asr_megakernel.py:767-773)."""
-        n = int(ids.numel())
-        if n > self.max_prefill_len_:
-            raise RuntimeError("Prefill sequence length exceeds maximum")
-        if n == 0:
-            raise RuntimeError("Empty input sequence")
-        if pos0 + n > self.max_seq_len_:
-            raise RuntimeError("Prefill sequence length exceeds maximum (max_seq_len)")
-        return n
 
     def prefill_step(self, input_ids) -> int:
         """Full-sequence forward from position 0: afterwards ``position() == len(ids)``

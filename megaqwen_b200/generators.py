@@ -8,22 +8,17 @@ from __future__ import annotations
 
 import torch
 
-from .decoder import MegakernelDecoder
-from .weights import load_qwen3_weights
+from .registry import build_decoder
 
 
 class MegakernelGenerator:
     """Decode-only generator: the prompt is fed one token at a time through
     ``decode_step`` (reference: megakernel_generators.py:12-63).  Greedy;
-    ``temperature`` is accepted and ignored, as in the reference."""
+    ``temperature`` is accepted and ignored, as in the reference.  ``model_name``
+    may be a directory of any registered model (registry.py)."""
 
-    def __init__(self, model_name="Qwen/Qwen3-0.6B", max_seq_len=2048, weights=None, device="cuda"):
-        weights = weights or load_qwen3_weights(model_name, max_seq_len=max_seq_len, device=device)
-        self.decoder = MegakernelDecoder(
-            weights["embed_weight"], weights["layer_weights"], weights["final_norm_weight"],
-            weights["lm_head_weight"], weights["cos_table"], weights["sin_table"],
-            len(weights["layer_weights"]) // 11, max_seq_len, max_seq_len)
-        self.tokenizer = weights.get("tokenizer")
+    def __init__(self, model_name="Qwen/Qwen3-0.6B", max_seq_len=2048, weights=None, device="cuda", dtype="bfloat16"):
+        self.decoder, self.tokenizer = build_decoder(model_name, max_seq_len, weights=weights, dtype=dtype, device=device)
         self.max_seq_len = max_seq_len
 
     def _stops(self, stop_tokens):
@@ -69,8 +64,9 @@ class MegakernelPrefillGenerator(MegakernelGenerator):
     The stop token is excluded from the output; the first generated token is the
     one ``prefill_step`` returns."""
 
-    def __init__(self, model_name="Qwen/Qwen3-0.6B", max_seq_len=2048, max_prefill_len=512, weights=None, device="cuda"):
-        super().__init__(model_name, max_seq_len, weights=weights, device=device)
+    def __init__(self, model_name="Qwen/Qwen3-0.6B", max_seq_len=2048, max_prefill_len=512, weights=None, device="cuda",
+                 dtype="bfloat16"):
+        super().__init__(model_name, max_seq_len, weights=weights, device=device, dtype=dtype)
         self.decoder.max_prefill_len_ = max_prefill_len
         self.max_prefill_len = max_prefill_len
 

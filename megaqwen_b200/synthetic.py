@@ -13,7 +13,7 @@ from __future__ import annotations
 
 import torch
 
-from .spec import ModelSpec
+from .spec import HybridSpec, ModelSpec
 
 
 def rope_tables(max_seq_len: int, rope_theta: float, head_dim: int, device="cpu"):
@@ -56,7 +56,24 @@ def random_weights(spec: ModelSpec, max_seq_len: int, seed: int = 0, device="cpu
     }
 
 
-def random_prompt(spec: ModelSpec, length: int, cfg_idx: int = 1, seq_idx: int = 0) -> torch.Tensor:
+def random_hybrid_weights(spec: HybridSpec, seed: int = 0, device="cpu") -> dict:
+    """Checkpoint tensors of a layer-listed model by name: matrices randn / sqrt(inputs), drawn in the order
+    of ``spec.tensor_shapes()`` from one generator; norms near their neutral value, sinks randn."""
+    g = torch.Generator().manual_seed(seed)
+    tensors = {}
+    for name, shape in spec.tensor_shapes().items():
+        t = torch.randn(shape, generator=g, dtype=torch.float32)
+        if len(shape) == 2:
+            t = t / (shape[1] ** 0.5 if name != "embed" else spec.embed_scale)
+        elif name.endswith(("mix.norm", "dkv.norm")):
+            t = 1.0 + 0.1 * t
+        elif not name.endswith("sink"):
+            t = 0.1 * t                      # stored around zero
+        tensors[name] = t.to(torch.bfloat16).to(device)
+    return {"spec": spec, "tensors": tensors, "tokenizer": None}
+
+
+def random_prompt(spec, length: int, cfg_idx: int = 1, seq_idx: int = 0) -> torch.Tensor:
     """Uniform random token ids, int32 [length], seed 1000 + 100*cfg + seq."""
     g = torch.Generator().manual_seed(1000 + cfg_idx * 100 + seq_idx)
     return torch.randint(0, spec.vocab_size, (length,), generator=g).to(torch.int32)

@@ -16,7 +16,7 @@ import os
 
 import torch
 
-from .spec import QWEN3_0_6B, QWEN3_TINY, ModelSpec
+from .spec import QWEN3_0_6B, QWEN3_TINY, ModelSpec, read_hybrid_config
 from .synthetic import random_weights, rope_tables
 
 _LAYER_KEYS = ["input_layernorm.weight", "self_attn.q_proj.weight", "self_attn.k_proj.weight",
@@ -65,6 +65,29 @@ def _bf16(t, device):
     return t.to(torch.bfloat16).contiguous().to(device)
 
 
+def load_tokenizer(model_dir: str):
+    """The tokenizer beside the weights, or None."""
+    try:
+        from transformers import AutoTokenizer
+        return AutoTokenizer.from_pretrained(model_dir, local_files_only=True)
+    except Exception:
+        return None
+
+
+def load_hybrid_weights(model_dir: str, max_seq_len: int = 2048, device="cuda") -> dict:
+    """Tensors of a layer-listed model by their checkpoint names (on the CPU: the decoder packs them on
+    ``device``), with the spec its config.json describes."""
+    with open(os.path.join(model_dir, "config.json")) as fh:
+        spec = read_hybrid_config(json.load(fh))
+    shapes = spec.tensor_shapes()
+    tensors = load_tensors(model_dir, list(shapes))
+    for name, shape in shapes.items():
+        if tuple(tensors[name].shape) != shape:
+            raise RuntimeError(f"{name}: config.json describes {shape}, the checkpoint holds {tuple(tensors[name].shape)}")
+    has_tokenizer = any(os.path.exists(os.path.join(model_dir, f)) for f in ("tokenizer.json", "tokenizer_config.json", "vocab.json"))
+    return {"spec": spec, "tensors": tensors, "tokenizer": load_tokenizer(model_dir) if has_tokenizer else None}
+
+
 def load_qwen3_weights(model_name="Qwen/Qwen3-0.6B", max_seq_len=2048, device="cuda", spec: ModelSpec | None = None, seed: int = 0) -> dict:
     if model_name in ("synthetic", "synthetic-tiny"):
         spec = spec or (QWEN3_TINY if model_name == "synthetic-tiny" else QWEN3_0_6B)
@@ -96,11 +119,6 @@ def load_qwen3_weights(model_name="Qwen/Qwen3-0.6B", max_seq_len=2048, device="c
     lm_head = embed if "lm_head.weight" not in t or cfg.get("tie_word_embeddings", True) else _bf16(t["lm_head.weight"], device)
     layer_weights = [_bf16(t[f"{prefix}layers.{l}.{k}"], device) for l in range(spec.num_layers) for k in _LAYER_KEYS]
     cos, sin = rope_tables(max_seq_len, spec.rope_theta, spec.head_dim, device)
-    tokenizer = None
-    try:
-        from transformers import AutoTokenizer
-        tokenizer = AutoTokenizer.from_pretrained(model_name, local_files_only=True)
-    except Exception:
-        tokenizer = None
+    tokenizer = load_tokenizer(model_name)
     return {"embed_weight": embed, "layer_weights": layer_weights, "final_norm_weight": _bf16(t[prefix + "norm.weight"], device),
             "lm_head_weight": lm_head, "cos_table": cos, "sin_table": sin, "tokenizer": tokenizer, "spec": spec}
