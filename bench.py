@@ -9,6 +9,7 @@ tokens/s through the public decoder API with host inputs and outputs
 `prefill_step(cpu ids)` is reported beside it.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference]
+    python bench.py --hybrid              # layer-listed models beside Qwen3-0.6B: prefill and decode throughput
 
 With --gpus N > 1 (under torchrun) every rank runs an independent replica on
 its own GPU with its own prompt; there is no data-path communication.
@@ -443,6 +444,102 @@ def run_ours(args):
     print(json.dumps(line))
 
 
+def hybrid_spec(name):
+    """Layer-listed models at the sizes of real ones (random weights): "0.6b" has the layers, width, heads and
+    vocabulary of Qwen3-0.6B, "0.6b-loop" half of its layers with a stretch that runs twice, "2b" wider layers."""
+    from megaqwen_b200.spec import HybridSpec, LayerSpec, MixerSpec
+    width, ff, layers, loop = {"0.6b": (1024, 3072, 28, None), "0.6b-loop": (1024, 3072, 14, (2, 12, 2)), "2b": (2048, 6144, 20, None)}[name]
+    latent = MixerSpec("latent_attention", 16, 128, 128, rank=512, rot=64, rot_base=1e6, scale=192 ** -0.5)
+    light = MixerSpec("lightning", 16, 128, 128, decay=tuple(1.0 - 2.0 ** (-1 - 0.5 * i) for i in range(16)))
+    return HybridSpec(vocab_size=151936, hidden_size=width, embed_scale=1.0, rms_eps=1e-6, residual_mult=0.2,
+                      layers=tuple(LayerSpec(light if i % 2 else latent, ff) for i in range(layers)), loop=loop)
+
+
+def measure_decoder(dec, dev, spec, peaks, vocab):
+    """Prefill of whole prompts and decode chains (graph replay) at several lengths, through the decoder's
+    public calls; CUDA events around the calls, best of a few."""
+    hbm, bf16 = peaks
+    g = torch.Generator().manual_seed(11)
+
+    def timed(fn, repeats):
+        best = 1e9
+        for _ in range(repeats):
+            torch.cuda.synchronize(dev)
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record(); fn(); e1.record()
+            torch.cuda.synchronize(dev)
+            best = min(best, e0.elapsed_time(e1))
+        return best
+
+    out = {"prefill": {}, "decode": {}}
+    for n in (128, 512, 1024, 2048):
+        ids = torch.randint(0, vocab, (n,), generator=g).to(torch.int32).to(dev)
+
+        def one():
+            dec.position_ = 0               # the states' contents do not change the work
+            dec.prefill_append(ids)
+        ms = timed(one, 6)
+        tf = spec.prefill_flops(n) / ms / 1e9
+        out["prefill"][str(n)] = {"ms": ms, "tokens_per_s": n / ms * 1e3, "tflops": tf, "frac_of_measured_bf16": tf / bf16}
+    for ctx in (16, 128, 512, 2048):
+        nbytes = sum(spec.decode_bytes(ctx + i) for i in range(32)) / 32
+
+        def chain():
+            dec.position_ = ctx - 1
+            dec._chain(17, 32, True)
+        chain()
+        us = timed(chain, 4) / 32 * 1e3
+        gbs = nbytes / us / 1e3
+        out["decode"][str(ctx)] = {"us_per_token": us, "tokens_per_s": 1e6 / us, "MB_per_token": nbytes / 1e6, "GBps": gbs, "frac_of_measured_hbm": gbs / hbm}
+    dec.check_status()
+    return out
+
+
+def run_hybrid(args):
+    """Layer-listed models beside the framework's other model at equal size; prints one JSON line."""
+    from megaqwen_b200.decoder import MegakernelDecoder
+    from megaqwen_b200.hybrid import HybridDecoder
+    from megaqwen_b200.synthetic import random_hybrid_weights
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    hbm, kind = load_peaks()
+    bf16 = 1590.0
+    if kind == "measured":
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as fh:
+            bf16 = float(json.load(fh)["bf16_tflops"])
+    sampler = ClockSampler(0)
+    sampler.start()
+    result = {}
+    for name in args.hybrid_sizes.split(","):
+        if name == "qwen3-0.6b":
+            w = random_weights(QWEN3_0_6B, MAX_SEQ)
+            embed = w["embed_weight"].to(dev)
+            dec = MegakernelDecoder(embed, [t.to(dev) for t in w["layer_weights"]], w["final_norm_weight"].to(dev), embed, w["cos_table"].to(dev),
+                                    w["sin_table"].to(dev), QWEN3_0_6B.num_layers, MAX_SEQ, PROMPT_LEN)
+            spec, vocab = QWEN3_0_6B, QWEN3_0_6B.vocab_size
+        else:
+            spec = hybrid_spec(name)
+            vocab = spec.vocab_size
+            dec = HybridDecoder(random_hybrid_weights(spec, device=dev), MAX_SEQ, PROMPT_LEN, device=dev)
+        if args.ncu_case > 0:               # profiler case: one prefill of --ncu-prefill tokens, or eager decode steps at --ncu-pos
+            if args.ncu_prefill > 0:
+                ids = torch.randint(0, vocab, (args.ncu_prefill,)).to(torch.int32)
+                for _ in range(args.ncu_case):
+                    dec.position_ = 0
+                    dec.prefill_append(ids)
+            else:
+                dec.position_ = args.ncu_pos
+                dec.decode_steps_cuda(17, args.ncu_case)
+            dec.check_status()
+            result[name] = {"launches": dec.launches}
+        else:
+            result[name] = measure_decoder(dec, dev, spec, (hbm, bf16), vocab)
+        del dec
+        torch.cuda.empty_cache()
+    print(json.dumps({"metric": "hybrid_prefill_and_decode", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic", "models": result,
+                      "peaks": {"hbm_gbs": hbm, "bf16_tflops": bf16, "kind": kind}, "clocks": sampler.stop()}))
+
+
 def run_ncu_case(args):
     """Small case for profiler captures: a few eager decode steps at context 2048
     over a cache filled with random values (no 2048-step prompt before them)."""
@@ -507,8 +604,12 @@ def main():
     ap.add_argument("--ncu-prefill", type=int, default=0, help="profiler case: N prefills of this many tokens instead of decode steps")
     ap.add_argument("--ncu-batch", type=int, default=0, help="profiler case: batched decode steps with this batch size")
     ap.add_argument("--ncu-persistent", action="store_true", help="profiler case runs the persistent chain kernel")
+    ap.add_argument("--hybrid", action="store_true", help="measure layer-listed models beside Qwen3-0.6B instead of the headline workload")
+    ap.add_argument("--hybrid-sizes", default="qwen3-0.6b,0.6b,0.6b-loop,2b", help="models of --hybrid, with commas between them")
     args = ap.parse_args()
-    if args.ncu_case > 0:
+    if args.hybrid:
+        run_hybrid(args)
+    elif args.ncu_case > 0:
         run_ncu_case(args)
     elif args.impl == "reference":
         run_reference(args)
