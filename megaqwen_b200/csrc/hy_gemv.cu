@@ -81,6 +81,11 @@ __global__ void __launch_bounds__(GV_THREADS, 2) k_gemv(GemvArgs a) {
     };
 #pragma unroll
     for (int d = 0; d < GV_D; ++d) load(ring[d]);
+    // The rest of the warp's rows is asked into the L2 at the same time.
+    if (lane == 0 && r1 > r0) {
+        const size_t ahead = (size_t)GV_D * ((CHUNK < K ? CHUNK : K)), total = (size_t)(r1 - r0) * K;
+        if (OUT != OUT_HEAD && total > ahead) l2_prefetch(W + (size_t)r0 * K + ahead, (uint32_t)((total - ahead) * sizeof(T)));
+    }
     if (OUT != OUT_HEAD) pdl_trigger();
     pdl_wait_cta();
     // The LM head lets the next step begin only now: every kernel of this step has completed, so that the step after
@@ -242,7 +247,9 @@ static int go(Stream& st, const GemvArgs& a) {
     const size_t smem = (size_t)((a.K + CHUNK - 1) / CHUNK) * CHUNK * sizeof(float);
     const int rc = allow_smem(k_gemv<T, VEC, OUT>, smem);
     if (rc) return rc;
-    return launch(st, k_gemv<T, VEC, OUT>, dim3(sm_count()), dim3(GV_THREADS), smem, a);
+    // The LM head is long enough to fill the device by itself: two CTAs per SM keep more loads in flight.  The products of
+    // a layer take one, so that the next kernel's CTA fits beside it.
+    return launch(st, k_gemv<T, VEC, OUT>, dim3(OUT == OUT_HEAD ? 2 * sm_count() : sm_count()), dim3(GV_THREADS), smem, a);
 }
 template <typename T>
 int gemv(Stream& st, int vec, int out, const GemvArgs& a) {

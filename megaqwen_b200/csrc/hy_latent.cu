@@ -28,6 +28,20 @@ __device__ __forceinline__ float2 load2(const bf16* p) {
 __device__ __forceinline__ void store2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
 __device__ __forceinline__ void store2(bf16* p, float2 v) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(v.x, v.y); }
 
+// acc + 16 bytes of a weight row times the vector elements at v
+__device__ __forceinline__ float dot_row16(const uint4& u, const float* v, float acc, const bf16*) {
+    const float4 a = load4(v), b = load4(v + 4);
+    acc = fmaf(bf_lo(u.x), a.x, acc); acc = fmaf(bf_hi(u.x), a.y, acc); acc = fmaf(bf_lo(u.y), a.z, acc); acc = fmaf(bf_hi(u.y), a.w, acc);
+    acc = fmaf(bf_lo(u.z), b.x, acc); acc = fmaf(bf_hi(u.z), b.y, acc); acc = fmaf(bf_lo(u.w), b.z, acc); acc = fmaf(bf_hi(u.w), b.w, acc);
+    return acc;
+}
+__device__ __forceinline__ float dot_row16(const uint4& u, const float* v, float acc, const float*) {
+    const float4 a = load4(v);
+    acc = fmaf(__uint_as_float(u.x), a.x, acc); acc = fmaf(__uint_as_float(u.y), a.y, acc);
+    acc = fmaf(__uint_as_float(u.z), a.z, acc); acc = fmaf(__uint_as_float(u.w), a.w, acc);
+    return acc;
+}
+
 // One cache row from the down projection of a token: c = rms(down[0, rank)) * norm, then the rotated key part.
 // NT threads of a CTA.
 template <typename T, int NT>
@@ -220,15 +234,7 @@ __global__ void __launch_bounds__(LQ_THREADS) k_latent_query(LatentDecodeArgs a)
         float s = 0.f;
         for (int c0 = ln * EPL; c0 < a.dim && ok; c0 += 32 * EPL) {     // one pass unless dim > 32 * EPL
             const uint4 u = c0 == ln * EPL ? w[x] : *reinterpret_cast<const uint4*>(W + (size_t)r * a.dim + c0);
-            if constexpr (EPL == 8) {
-                const float4 v0 = load4(lq_q + c0), v1 = load4(lq_q + c0 + 4);
-                s = fmaf(bf_lo(u.x), v0.x, s); s = fmaf(bf_hi(u.x), v0.y, s); s = fmaf(bf_lo(u.y), v0.z, s); s = fmaf(bf_hi(u.y), v0.w, s);
-                s = fmaf(bf_lo(u.z), v1.x, s); s = fmaf(bf_hi(u.z), v1.y, s); s = fmaf(bf_lo(u.w), v1.z, s); s = fmaf(bf_hi(u.w), v1.w, s);
-            } else {
-                const float4 v0 = load4(lq_q + c0);
-                s = fmaf(__uint_as_float(u.x), v0.x, s); s = fmaf(__uint_as_float(u.y), v0.y, s);
-                s = fmaf(__uint_as_float(u.z), v0.z, s); s = fmaf(__uint_as_float(u.w), v0.w, s);
-            }
+            s = dot_row16(u, lq_q + c0, s, (const T*)nullptr);
         }
         for (int o = lanes >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
         if (ok && ln == 0) qc[r] = Elem<T>::put(s);
@@ -247,7 +253,8 @@ __device__ __forceinline__ int keys_per_split(int ctx, int splits) {
     return ((tiles + splits - 1) / splits) * LA_KEYS;
 }
 __device__ __forceinline__ int clamp_pos(int pos, int max_seq) { return pos < 0 ? 0 : pos >= max_seq ? max_seq - 1 : pos; }
-// A split leaves behind, per head, the sum of its weighted latents [rank], their maximum and the sum of weights.
+// A split leaves behind, per head, the sum of its weighted latents (parts [split][head][rank]) and, after all of those, the
+// maximum of its scores and the sum of its weights (pairs [split][head]).
 size_t latent_parts_floats(int heads, int rank, int max_seq) { return (size_t)latent_splits(max_seq) * heads * (rank + 2); }
 
 // bf16, up to 512 latent dimensions: sixteen heads are the M of mma.sync, so every cached row is read once for all of them.
@@ -303,6 +310,7 @@ __global__ void __launch_bounds__(LA_THREADS) k_latent_attention(LatentDecodeArg
         const uint32_t qa = smem_u32(sq + (lane & 15) * ld + (lane >> 4) * 8);
         const uint32_t kb = smem_u32(sk + (warp * 8 + row) * ld + (lane & 3) * 2);
         int ks = 0;
+#pragma unroll 3
         for (; ks + 1 < D / 16; ks += 2) {
             uint32_t q4[4], r4[4];
             ldsm4(q4, qa + ks * 32);
@@ -370,18 +378,19 @@ __global__ void __launch_bounds__(LA_THREADS) k_latent_attention(LatentDecodeArg
         __syncthreads();                                   // keys, weights and maxima are overwritten by the next tile
     }
     const int heads_here = min(16, a.heads - h0);
-    float* part = a.parts + ((size_t)split * a.heads + h0) * (a.rank + 2);
+    const size_t part = (size_t)split * a.heads + h0;
+    float2* ml = reinterpret_cast<float2*>(a.parts + (size_t)gridDim.x * a.heads * a.rank);
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
         const int r = row + 8 * h;
         if (r >= heads_here) continue;
-        float* dst = part + (size_t)r * (a.rank + 2);
+        float* dst = a.parts + (part + r) * a.rank;
 #pragma unroll
         for (int i = 0; i < LA_MAXT; ++i) {
             if (i >= tpw || tile0 + i >= ntiles) break;
             *reinterpret_cast<float2*>(dst + (tile0 + i) * 8 + 2 * (lane & 3)) = make_float2(acc[i][2 * h], acc[i][2 * h + 1]);
         }
-        if (warp == 0 && (lane & 3) == 0) *reinterpret_cast<float2*>(dst + a.rank) = make_float2(m[h], l[h]);
+        if (warp == 0 && (lane & 3) == 0) ml[part + r] = make_float2(m[h], l[h]);
     }
 }
 
@@ -434,24 +443,29 @@ __global__ void __launch_bounds__(LP_THREADS) k_latent_attention_plain(LatentDec
         }
         __syncthreads();
     }
-    float* dst = a.parts + ((size_t)split * a.heads + head) * (a.rank + 2);
+    const size_t part = (size_t)split * a.heads + head;
+    float* dst = a.parts + part * a.rank;
 #pragma unroll
     for (int x = 0; x < LP_MAXC; ++x) {
         const int i = tid + x * LP_THREADS;
         if (i < a.rank) dst[i] = acc[x];
     }
-    if (tid == 0) { dst[a.rank] = m; dst[a.rank + 1] = l; }
+    if (tid == 0) reinterpret_cast<float2*>(a.parts + (size_t)gridDim.x * a.heads * a.rank)[part] = make_float2(m, l);
 }
 
 // ---------------------------------------------------------------- one token: merge
 // CTA (x, h): the latent sum of head h over all splits, the sink in the denominator, then rows [32 x, 32 x + 32) of its W_uv.
+// Thread = (group of splits, four latent columns); the groups' sums meet in shared memory.
 constexpr int LM_ROWS = 32, LM_THREADS = 256, LM_PRE = 2;
+static __host__ __device__ __forceinline__ int lm_groups(int rank) { return rank >= 4 * LM_THREADS ? 1 : 4 * LM_THREADS / rank < 8 ? 4 * LM_THREADS / rank : 8; }
 template <typename T>
 __global__ void __launch_bounds__(LM_THREADS) k_latent_merge(LatentDecodeArgs a, int splits) {
-    extern __shared__ float lm_c[];                        // [rank], then the weight of every split
+    extern __shared__ float lm_c[];                        // [groups][rank], then the weight of every split
+    __shared__ float red[8];
     constexpr int EPL = Elem<T>::PER16;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y;
-    float* ws = lm_c + a.rank;
+    const int groups = lm_groups(a.rank), cols = a.rank / 4;
+    float* ws = lm_c + groups * a.rank;
     const int r0 = blockIdx.x * LM_ROWS + warp * (LM_ROWS / 8);
     const T* W = reinterpret_cast<const T*>(a.w_uv) + (size_t)h * a.vdim * a.rank;
     uint4 w[LM_ROWS / 8][LM_PRE];
@@ -465,48 +479,54 @@ __global__ void __launch_bounds__(LM_THREADS) k_latent_merge(LatentDecodeArgs a,
     pdl_trigger();
     pdl_wait_cta();
     const int ctx = clamp_pos(*a.position, a.max_seq) + 1;
-    const int kps = keys_per_split(ctx, splits), active = (ctx + kps - 1) / kps;
-    const float* part = a.parts + (size_t)h * (a.rank + 2);
-    const size_t stride = (size_t)a.heads * (a.rank + 2);
-    for (int s = tid; s < active; s += LM_THREADS) ws[s] = __ldcg(part + s * stride + a.rank);
-    __syncthreads();
+    const int kps = keys_per_split(ctx, splits), active = (ctx + kps - 1) / kps;      // at most 148 < LM_THREADS
+    const size_t hs = (size_t)h, stride = (size_t)a.heads;
+    const float2* ml = reinterpret_cast<const float2*>(a.parts + (size_t)splits * a.heads * a.rank);
     const float sink = a.sink ? a.sink[h] * LOG2E : -INFINITY;
-    float m = sink;
-    for (int s = 0; s < active; ++s) m = fmaxf(m, ws[s]);
+    const float2 mine = tid < active ? __ldcg(ml + tid * stride + hs) : make_float2(-INFINITY, 0.f);
+    float m = warp_max(mine.x);
+    if (lane == 0) red[warp] = m;
     __syncthreads();
-    float l = 0.f;
-    for (int s = tid; s < active; s += LM_THREADS) {
-        const float e = exp2f(ws[s] - m);
-        l += e * __ldcg(part + s * stride + a.rank + 1);
-        ws[s] = e;
-    }
-    __shared__ float red[8];
-    const float inv = 1.0f / (cta_sum<8>(l, red) + exp2f(sink - m));
-    for (int i = tid; i < a.rank; i += LM_THREADS) {
-        float s = 0.f;
+    m = sink;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) m = fmaxf(m, red[i]);
+    __syncthreads();
+    const float e = exp2f(mine.x - m);
+    if (tid < active) ws[tid] = e;
+    const float inv = 1.0f / (cta_sum<8>(e * mine.y, red) + exp2f(sink - m));
+    for (int x = tid; x < groups * cols; x += LM_THREADS) {
+        const int g = x / cols, c = (x % cols) * 4;
+        const float* p = a.parts + hs * a.rank + c;
+        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
-        for (int x = 0; x < active; ++x) s = fmaf(ws[x], __ldcg(part + x * stride + i), s);
-        lm_c[i] = s * inv;
+        for (int k = g; k < active; k += groups) {
+            const float4 v = load4_cg(p + k * stride * a.rank);
+            const float f = ws[k];
+            s.x = fmaf(f, v.x, s.x); s.y = fmaf(f, v.y, s.y); s.z = fmaf(f, v.z, s.z); s.w = fmaf(f, v.w, s.w);
+        }
+        store4(lm_c + g * a.rank + c, make_float4(s.x * inv, s.y * inv, s.z * inv, s.w * inv));
     }
     __syncthreads();
+    if (groups > 1) {
+        for (int i = tid; i < a.rank; i += LM_THREADS) {
+            float s = lm_c[i];
+            for (int g = 1; g < groups; ++g) s += lm_c[g * a.rank + i];
+            lm_c[i] = s;
+        }
+        __syncthreads();
+    }
 #pragma unroll
     for (int x = 0; x < LM_ROWS / 8; ++x) {
         const int r = r0 + x;
         if (r >= a.vdim) break;
         float s = 0.f;
-        int seg = 0;
-        for (int c0 = lane * EPL; c0 < a.rank; c0 += 32 * EPL, ++seg) {
-            const uint4 u = seg == 0 ? w[x][0] : seg == 1 ? w[x][1] : *reinterpret_cast<const uint4*>(W + (size_t)r * a.rank + c0);
-            if constexpr (EPL == 8) {
-                const float4 v0 = load4(lm_c + c0), v1 = load4(lm_c + c0 + 4);
-                s = fmaf(bf_lo(u.x), v0.x, s); s = fmaf(bf_hi(u.x), v0.y, s); s = fmaf(bf_lo(u.y), v0.z, s); s = fmaf(bf_hi(u.y), v0.w, s);
-                s = fmaf(bf_lo(u.z), v1.x, s); s = fmaf(bf_hi(u.z), v1.y, s); s = fmaf(bf_lo(u.w), v1.z, s); s = fmaf(bf_hi(u.w), v1.w, s);
-            } else {
-                const float4 v0 = load4(lm_c + c0);
-                s = fmaf(__uint_as_float(u.x), v0.x, s); s = fmaf(__uint_as_float(u.y), v0.y, s);
-                s = fmaf(__uint_as_float(u.z), v0.z, s); s = fmaf(__uint_as_float(u.w), v0.w, s);
-            }
+#pragma unroll
+        for (int seg = 0; seg < LM_PRE; ++seg) {
+            const int c0 = (seg * 32 + lane) * EPL;
+            if (c0 < a.rank) s = dot_row16(w[x][seg], lm_c + c0, s, (const T*)nullptr);
         }
+        for (int c0 = (LM_PRE * 32 + lane) * EPL; c0 < a.rank; c0 += 32 * EPL)
+            s = dot_row16(*reinterpret_cast<const uint4*>(W + (size_t)r * a.rank + c0), lm_c + c0, s, (const T*)nullptr);
         s = warp_sum(s);
         if (lane == 0) reinterpret_cast<T*>(a.out)[(size_t)h * a.vdim + r] = Elem<T>::put(s);
     }
@@ -527,7 +547,7 @@ int latent_decode(Stream& st, const LatentDecodeArgs& a) {
         rc = launch(st, k_latent_attention_plain<T>, dim3(splits, a.heads), dim3(LP_THREADS), (size_t)D * 4, a);
     }
     if (rc) return rc;
-    return launch(st, k_latent_merge<T>, dim3((a.vdim + LM_ROWS - 1) / LM_ROWS, a.heads), dim3(LM_THREADS), (size_t)(a.rank + splits) * 4, a, splits);
+    return launch(st, k_latent_merge<T>, dim3((a.vdim + LM_ROWS - 1) / LM_ROWS, a.heads), dim3(LM_THREADS), (size_t)(lm_groups(a.rank) * a.rank + splits) * 4, a, splits);
 }
 template int latent_decode<bf16>(Stream&, const LatentDecodeArgs&);
 template int latent_decode<float>(Stream&, const LatentDecodeArgs&);
