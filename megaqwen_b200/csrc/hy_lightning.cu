@@ -160,10 +160,9 @@ __global__ void __launch_bounds__(LK_THREADS) k_lightning_kv(LightningArgs a, fl
 }
 
 // ---------------------------------------------------------------- chunked: the state before every chunk
-// Element by element over the chunks: planes[c] = state (two bf16 terms, in place of the chunk's KV: eight bytes become
-// eight), state <- decay^n state + KV.
+// Element by element over the chunks: hi[c], lo[c] = the two bf16 terms of the state, state <- decay^n state + KV[c].
 constexpr int LN_THREADS = 128, LN_AHEAD = 8;
-__global__ void __launch_bounds__(LN_THREADS) k_lightning_scan(LightningArgs a, float* __restrict__ kv) {
+__global__ void __launch_bounds__(LN_THREADS) k_lightning_scan(LightningArgs a, const float* __restrict__ kv, bf16* __restrict__ hi, bf16* __restrict__ lo) {
     pdl_trigger();
     const size_t e = ((size_t)blockIdx.x * LN_THREADS + threadIdx.x) * 4, plane = (size_t)a.heads * a.dim * a.vdim;
     const bool live = e < plane;
@@ -181,10 +180,11 @@ __global__ void __launch_bounds__(LN_THREADS) k_lightning_scan(LightningArgs a, 
 #pragma unroll
         for (int x = 0; x < LN_AHEAD; ++x)
             if (c0 + x < nchunks) {
-                uint4 o;                                       // hi, lo of elements 0, 1, then of 2, 3
-                split_pair(s.x, s.y, o.x, o.y);
-                split_pair(s.z, s.w, o.z, o.w);
-                *reinterpret_cast<uint4*>(kv + (c0 + x) * plane + e) = o;
+                uint2 h, l;
+                split_pair(s.x, s.y, h.x, l.x);
+                split_pair(s.z, s.w, h.y, l.y);
+                *reinterpret_cast<uint2*>(hi + (c0 + x) * plane + e) = h;
+                *reinterpret_cast<uint2*>(lo + (c0 + x) * plane + e) = l;
                 const float d = c0 + x == nchunks - 1 ? last : full;
                 s.x = fmaf(d, s.x, v[x].x); s.y = fmaf(d, s.y, v[x].y); s.z = fmaf(d, s.z, v[x].z); s.w = fmaf(d, s.w, v[x].w);
             }
@@ -197,7 +197,7 @@ __global__ void __launch_bounds__(LN_THREADS) k_lightning_scan(LightningArgs a, 
 // o_t = decay^(t + 1) q_t S + sum over s <= t of (q_t k_s) decay^(t - s) v_s      (t, s within the chunk)
 constexpr int LO_THREADS = 128;
 static size_t lo_smem(int dim) { return ((size_t)(64 + LC) * (dim + 8) + (size_t)LC * LO_VLD + (size_t)2 * dim * LO_VLD) * 2; }
-__global__ void __launch_bounds__(LO_THREADS) k_lightning_out(LightningArgs a, const uint32_t* __restrict__ states) {
+__global__ void __launch_bounds__(LO_THREADS) k_lightning_out(LightningArgs a, const bf16* __restrict__ hi, const bf16* __restrict__ lo) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) uint8_t lo_raw[];
@@ -216,12 +216,18 @@ __global__ void __launch_bounds__(LO_THREADS) k_lightning_out(LightningArgs a, c
     const bf16* qg = reinterpret_cast<const bf16*>(a.q) + row0 * ldk + (size_t)head * dim;
     const bf16* kg = reinterpret_cast<const bf16*>(a.k) + row0 * ldk + (size_t)head * dim;
     const bf16* vg = reinterpret_cast<const bf16*>(a.v) + row0 * ldv + (size_t)head * vdim + j0;
-    const uint32_t* sg = states + ((size_t)c * a.heads + head) * dim * vdim + j0;
+    const size_t plane = ((size_t)c * a.heads + head) * dim * vdim + j0;
     const int dv8 = dim / 8;
     for (int x = tid; x < 64 * dv8; x += LO_THREADS) {
         const int t = x / dv8, col = (x % dv8) * 8;
         const bool ok = q0 + t < cnt;
         cp_async16_zfill(sq + t * qld + col, ok ? qg + (q0 + t) * ldk + col : qg, ok);
+    }
+    for (int x = tid; x < dim * 8; x += LO_THREADS) {
+        const int i = x >> 3, col = (x & 7) * 8;
+        const bool ok = j0 + col < vdim;
+        cp_async16_zfill(sh + i * LO_VLD + col, ok ? hi + plane + (size_t)i * vdim + col : hi, ok);
+        cp_async16_zfill(sl + i * LO_VLD + col, ok ? lo + plane + (size_t)i * vdim + col : lo, ok);
     }
     cp_async_commit();
     for (int x = tid; x < nkeys * dv8; x += LO_THREADS) {
@@ -235,23 +241,6 @@ __global__ void __launch_bounds__(LO_THREADS) k_lightning_out(LightningArgs a, c
         cp_async16_zfill(sv + t * LO_VLD + col, ok ? vg + t * ldv + col : vg, ok);
     }
     cp_async_commit();
-    // the state's terms come interleaved (see k_lightning_scan) and go to two planes
-    for (int x = tid; x < dim * 16; x += 4 * LO_THREADS) {
-        uint4 u[4];
-#pragma unroll
-        for (int y = 0; y < 4; ++y) {
-            const int i = (x + y * LO_THREADS) >> 4, col = ((x + y * LO_THREADS) & 15) * 4;
-            u[y] = i < dim && j0 + col < vdim ? ld_cg_u4(sg + (size_t)i * vdim + col) : make_uint4(0u, 0u, 0u, 0u);
-        }
-#pragma unroll
-        for (int y = 0; y < 4; ++y) {
-            const int i = (x + y * LO_THREADS) >> 4, col = ((x + y * LO_THREADS) & 15) * 4;
-            if (i < dim) {
-                *reinterpret_cast<uint2*>(sh + i * LO_VLD + col) = make_uint2(u[y].x, u[y].z);
-                *reinterpret_cast<uint2*>(sl + i * LO_VLD + col) = make_uint2(u[y].y, u[y].w);
-            }
-        }
-    }
     for (int i = tid; i <= LC; i += LO_THREADS) pw[i] = a.decay_pow[head * (LC + 1) + i];
     cp_async_wait<1>();
     __syncthreads();
@@ -336,18 +325,20 @@ __global__ void __launch_bounds__(LO_THREADS) k_lightning_out(LightningArgs a, c
     }
 }
 
-size_t lightning_scratch_bytes(int n, int heads, int dim, int vdim) { return (size_t)((n + LC - 1) / LC) * heads * dim * vdim * sizeof(float); }
+size_t lightning_scratch_bytes(int n, int heads, int dim, int vdim) { return (size_t)((n + LC - 1) / LC) * heads * dim * vdim * (sizeof(float) + 2 * sizeof(bf16)); }
 bool lightning_chunked_fits(int dim) { return lo_smem(dim) + (LC + 1) * 4 + 64 <= 232448 && lk_smem(dim) + LC * 4 + 64 <= 232448; }
 int lightning_chunked(Stream& st, const LightningArgs& a) {
     if (!lightning_chunked_fits(a.dim) || !a.scratch) return MQ_ERR_UNSUPPORTED;
     const int nchunks = (a.n + LC - 1) / LC, jt = (a.vdim + 63) / 64;
+    const size_t elems = (size_t)nchunks * a.heads * a.dim * a.vdim;
     float* kv = reinterpret_cast<float*>(a.scratch);
+    bf16 *hi = reinterpret_cast<bf16*>(kv + elems), *lo = hi + elems;
     int rc = allow_smem(k_lightning_kv, lk_smem(a.dim));
     if (!rc) rc = launch(st, k_lightning_kv, dim3(nchunks, a.heads, jt), dim3(LK_THREADS), lk_smem(a.dim), a, kv);
     const size_t quads = (size_t)a.heads * a.dim * a.vdim / 4;
-    if (!rc) rc = launch(st, k_lightning_scan, dim3((unsigned)((quads + LN_THREADS - 1) / LN_THREADS)), dim3(LN_THREADS), 0, a, kv);
+    if (!rc) rc = launch(st, k_lightning_scan, dim3((unsigned)((quads + LN_THREADS - 1) / LN_THREADS)), dim3(LN_THREADS), 0, a, (const float*)kv, hi, lo);
     if (!rc) rc = allow_smem(k_lightning_out, lo_smem(a.dim));
-    if (!rc) rc = launch(st, k_lightning_out, dim3(2 * nchunks, a.heads, jt), dim3(LO_THREADS), lo_smem(a.dim), a, (const uint32_t*)kv);
+    if (!rc) rc = launch(st, k_lightning_out, dim3(2 * nchunks, a.heads, jt), dim3(LO_THREADS), lo_smem(a.dim), a, (const bf16*)hi, (const bf16*)lo);
     return rc;
 }
 
