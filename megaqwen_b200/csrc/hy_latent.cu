@@ -42,25 +42,32 @@ __device__ __forceinline__ float dot_row16(const uint4& u, const float* v, float
     return acc;
 }
 
-// One cache row from the down projection of a token: c = rms(down[0, rank)) * norm, then the rotated key part.
-// NT threads of a CTA.
+// The latent of a token from its down projection: c = rms(down[0, rank)) * norm.  NT threads of a CTA; nw: the norm weights
+// of the thread's first two pairs, loaded ahead.
 template <typename T, int NT>
-__device__ __forceinline__ void write_cache_row(const float* down, const float* norm, int norm_n, float eps, const float* rope_row, T* row, int rank,
-                                                int rot, float* red) {
+__device__ __forceinline__ void write_latent(const float* down, const float* norm, const float2 (&nw)[2], int norm_n, float eps, T* row, int rank, float* red) {
     const int tid = threadIdx.x;
+    float2 keep[2];
     float ss = 0.f;
-    for (int i = tid * 2; i < rank; i += 2 * NT) {
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+        const int i = 2 * (tid + x * NT);
+        keep[x] = i < rank ? load2(down + i) : make_float2(0.f, 0.f);
+        ss += keep[x].x * keep[x].x + keep[x].y * keep[x].y;
+    }
+    for (int i = 2 * (tid + 2 * NT); i < rank; i += 2 * NT) {
         const float2 v = load2(down + i);
         ss += v.x * v.x + v.y * v.y;
     }
     const float inv = 1.0f / sqrtf(cta_sum<NT / 32>(ss, red) / (float)norm_n + eps);
-    for (int i = tid * 2; i < rank; i += 2 * NT) {
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+        const int i = 2 * (tid + x * NT);
+        if (i < rank) store2(row + i, make_float2(keep[x].x * inv * nw[x].x, keep[x].y * inv * nw[x].y));
+    }
+    for (int i = 2 * (tid + 2 * NT); i < rank; i += 2 * NT) {
         const float2 v = load2(down + i);
         store2(row + i, make_float2(v.x * inv * norm[i], v.y * inv * norm[i + 1]));
-    }
-    for (int i = tid; i < rot / 2; i += NT) {
-        const float2 v = load2(down + rank + 2 * i);
-        store2(row + rank + 2 * i, rotate_pair(v.x, v.y, reinterpret_cast<const float2*>(rope_row)[i]));
     }
 }
 
@@ -68,17 +75,29 @@ __device__ __forceinline__ void write_cache_row(const float* down, const float* 
 template <typename T>
 __global__ void __launch_bounds__(128) k_latent_rows(LatentRowsArgs a) {
     pdl_trigger();
-    pdl_wait();
     __shared__ float red[4];
-    const int t = blockIdx.x, pos = a.pos0 + t, D = a.rank + a.rot;
-    const float* rope = a.rope + (size_t)pos * a.rot;
-    T* q = reinterpret_cast<T*>(a.q_rot) + (size_t)t * a.heads * a.rot;
-    const int half = a.rot / 2;
-    for (int x = threadIdx.x; x < a.heads * half; x += 128) {
-        const float2 v = load2(q + 2 * x);
-        store2(q + 2 * x, rotate_pair(v.x, v.y, reinterpret_cast<const float2*>(rope)[x % half]));
+    const int t = blockIdx.x, tid = threadIdx.x, pos = a.pos0 + t, D = a.rank + a.rot;
+    const float2* rope = reinterpret_cast<const float2*>(a.rope + (size_t)pos * a.rot);
+    float2 nw[2];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+        const int i = 2 * (tid + x * 128);
+        nw[x] = i < a.rank ? *reinterpret_cast<const float2*>(a.norm + i) : make_float2(0.f, 0.f);
     }
-    write_cache_row<T, 128>(a.down + (size_t)t * D, a.norm, a.norm_n, a.eps, rope, reinterpret_cast<T*>(a.cache) + (size_t)pos * D, a.rank, a.rot, red);
+    pdl_wait();
+    T* q = reinterpret_cast<T*>(a.q_rot) + (size_t)t * a.heads * a.rot;
+    T* row = reinterpret_cast<T*>(a.cache) + (size_t)pos * D;
+    const float* down = a.down + (size_t)t * D;
+    const int half = a.rot / 2;
+    for (int x = tid; x < a.heads * half; x += 128) {
+        const float2 v = load2(q + 2 * x);
+        store2(q + 2 * x, rotate_pair(v.x, v.y, rope[x % half]));
+    }
+    for (int i = tid; i < half; i += 128) {
+        const float2 v = load2(down + a.rank + 2 * i);
+        store2(row + a.rank + 2 * i, rotate_pair(v.x, v.y, rope[i]));
+    }
+    write_latent<T, 128>(down, a.norm, nw, a.norm_n, a.eps, row, a.rank, red);
 }
 template <typename T>
 int latent_rows(Stream& st, const LatentRowsArgs& a) {
@@ -206,23 +225,40 @@ __global__ void __launch_bounds__(LQ_THREADS) k_latent_query(LatentDecodeArgs a)
             w[x] = ok ? *reinterpret_cast<const uint4*>(W + (size_t)r * a.dim + ln * EPL) : make_uint4(0u, 0u, 0u, 0u);
         }
     }
-    pdl_trigger();
-    pdl_wait_cta();
     if (extra) {
+        // what does not come from the kernel before is loaded before the wait (the position was set before this step began)
         int pos = *a.position;
         if (pos < 0 || pos >= a.max_seq) {
             if (tid == 0) atomicOr(a.status, MQ_STATUS_BAD_POSITION);
             pos = pos < 0 ? 0 : a.max_seq - 1;
         }
-        const float* rope = a.rope + (size_t)pos * a.rot;
-        const T* qr = reinterpret_cast<const T*>(a.q_rot) + (size_t)h * a.rot;
-        for (int i = tid; i < a.rot / 2; i += LQ_THREADS) {
-            const float2 v = load2(qr + 2 * i);
-            store2(qc + a.rank + 2 * i, rotate_pair(v.x, v.y, reinterpret_cast<const float2*>(rope)[i]));
+        const float2* rope = reinterpret_cast<const float2*>(a.rope + (size_t)pos * a.rot);
+        const int pairs = a.rot / 2;
+        float2 cs = tid < pairs ? rope[tid] : make_float2(1.f, 0.f);
+        float2 nw[2];
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+            const int i = 2 * (tid + x * LQ_THREADS);
+            nw[x] = h == 0 && i < a.rank ? *reinterpret_cast<const float2*>(a.norm + i) : make_float2(0.f, 0.f);
         }
-        if (h == 0) write_cache_row<T, LQ_THREADS>(a.down, a.norm, a.norm_n, a.eps, rope, reinterpret_cast<T*>(a.cache) + (size_t)pos * D, a.rank, a.rot, red);
+        pdl_trigger();
+        pdl_wait_cta();
+        const T* qr = reinterpret_cast<const T*>(a.q_rot) + (size_t)h * a.rot;
+        T* row = reinterpret_cast<T*>(a.cache) + (size_t)pos * D;
+        for (int i = tid; i < pairs; i += LQ_THREADS) {
+            if (i != tid) cs = rope[i];
+            const float2 q = load2(qr + 2 * i);
+            if (h == 0) {
+                const float2 k = load2(a.down + a.rank + 2 * i);
+                store2(row + a.rank + 2 * i, rotate_pair(k.x, k.y, cs));
+            }
+            store2(qc + a.rank + 2 * i, rotate_pair(q.x, q.y, cs));
+        }
+        if (h == 0) write_latent<T, LQ_THREADS>(a.down, a.norm, nw, a.norm_n, a.eps, row, a.rank, red);
         return;
     }
+    pdl_trigger();
+    pdl_wait_cta();
     const T* q = reinterpret_cast<const T*>(a.q) + (size_t)h * a.dim;
     for (int i = tid; i < a.dim; i += LQ_THREADS) lq_q[i] = Elem<T>::get(__ldcg(q + i));
     __syncthreads();
@@ -456,7 +492,7 @@ __global__ void __launch_bounds__(LP_THREADS) k_latent_attention_plain(LatentDec
 // ---------------------------------------------------------------- one token: merge
 // CTA (x, h): the latent sum of head h over all splits, the sink in the denominator, then rows [32 x, 32 x + 32) of its W_uv.
 // Thread = (group of splits, four latent columns); the groups' sums meet in shared memory.
-constexpr int LM_ROWS = 32, LM_THREADS = 256, LM_PRE = 2;
+constexpr int LM_ROWS = 32, LM_THREADS = 256, LM_PRE = 2, LM_FIRST = 8;
 static __host__ __device__ __forceinline__ int lm_groups(int rank) { return rank >= 4 * LM_THREADS ? 1 : 4 * LM_THREADS / rank < 8 ? 4 * LM_THREADS / rank : 8; }
 template <typename T>
 __global__ void __launch_bounds__(LM_THREADS) k_latent_merge(LatentDecodeArgs a, int splits) {
@@ -476,11 +512,18 @@ __global__ void __launch_bounds__(LM_THREADS) k_latent_merge(LatentDecodeArgs a,
             const int c0 = (s * 32 + lane) * EPL;
             w[x][s] = r0 + x < a.vdim && c0 < a.rank ? *reinterpret_cast<const uint4*>(W + (size_t)(r0 + x) * a.rank + c0) : make_uint4(0u, 0u, 0u, 0u);
         }
-    pdl_trigger();
-    pdl_wait_cta();
-    const int ctx = clamp_pos(*a.position, a.max_seq) + 1;
+    const int ctx = clamp_pos(*a.position, a.max_seq) + 1;                            // the position was set before this step began
     const int kps = keys_per_split(ctx, splits), active = (ctx + kps - 1) / kps;      // at most 148 < LM_THREADS
     const size_t hs = (size_t)h, stride = (size_t)a.heads;
+    pdl_trigger();
+    pdl_wait_cta();
+    // the first latent sums are on their way while the weights are worked out
+    float4 first[LM_FIRST];
+#pragma unroll
+    for (int y = 0; y < LM_FIRST; ++y) {
+        const int k = tid / cols + y * groups;
+        first[y] = tid < groups * cols && k < active ? load4_cg(a.parts + (k * stride + hs) * a.rank + (tid % cols) * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
     const float2* ml = reinterpret_cast<const float2*>(a.parts + (size_t)splits * a.heads * a.rank);
     const float sink = a.sink ? a.sink[h] * LOG2E : -INFINITY;
     const float2 mine = tid < active ? __ldcg(ml + tid * stride + hs) : make_float2(-INFINITY, 0.f);
@@ -498,12 +541,18 @@ __global__ void __launch_bounds__(LM_THREADS) k_latent_merge(LatentDecodeArgs a,
         const int g = x / cols, c = (x % cols) * 4;
         const float* p = a.parts + hs * a.rank + c;
         float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
-        for (int k = g; k < active; k += groups) {
-            const float4 v = load4_cg(p + k * stride * a.rank);
+        auto add = [&](int k, const float4& v) {
             const float f = ws[k];
             s.x = fmaf(f, v.x, s.x); s.y = fmaf(f, v.y, s.y); s.z = fmaf(f, v.z, s.z); s.w = fmaf(f, v.w, s.w);
+        };
+        int k = g;
+        if (x == tid) {
+#pragma unroll
+            for (int y = 0; y < LM_FIRST; ++y, k += groups)
+                if (k < active) add(k, first[y]);
         }
+#pragma unroll 8
+        for (; k < active; k += groups) add(k, load4_cg(p + k * stride * a.rank));
         store4(lm_c + g * a.rank + c, make_float4(s.x * inv, s.y * inv, s.z * inv, s.w * inv));
     }
     __syncthreads();
