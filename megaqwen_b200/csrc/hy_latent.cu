@@ -492,21 +492,21 @@ __global__ void __launch_bounds__(LP_THREADS) k_latent_attention_plain(LatentDec
 // ---------------------------------------------------------------- one token: merge
 // CTA (x, h): the latent sum of head h over all splits, the sink in the denominator, then rows [32 x, 32 x + 32) of its W_uv.
 // Thread = (group of splits, four latent columns); the groups' sums meet in shared memory.
-constexpr int LM_ROWS = 32, LM_THREADS = 256, LM_PRE = 2, LM_FIRST = 8;
+constexpr int LM_ROWS = 32, LM_THREADS = 512, LM_WARPS = LM_THREADS / 32, LM_PRE = 2, LM_FIRST = 8;
 static __host__ __device__ __forceinline__ int lm_groups(int rank) { return rank >= 4 * LM_THREADS ? 1 : 4 * LM_THREADS / rank < 8 ? 4 * LM_THREADS / rank : 8; }
 template <typename T>
 __global__ void __launch_bounds__(LM_THREADS) k_latent_merge(LatentDecodeArgs a, int splits) {
     extern __shared__ float lm_c[];                        // [groups][rank], then the weight of every split
-    __shared__ float red[8];
+    __shared__ float red[LM_WARPS];
     constexpr int EPL = Elem<T>::PER16;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y;
     const int groups = lm_groups(a.rank), cols = a.rank / 4;
     float* ws = lm_c + groups * a.rank;
-    const int r0 = blockIdx.x * LM_ROWS + warp * (LM_ROWS / 8);
+    const int r0 = blockIdx.x * LM_ROWS + warp * (LM_ROWS / LM_WARPS);
     const T* W = reinterpret_cast<const T*>(a.w_uv) + (size_t)h * a.vdim * a.rank;
-    uint4 w[LM_ROWS / 8][LM_PRE];
+    uint4 w[LM_ROWS / LM_WARPS][LM_PRE];
 #pragma unroll
-    for (int x = 0; x < LM_ROWS / 8; ++x)
+    for (int x = 0; x < LM_ROWS / LM_WARPS; ++x)
 #pragma unroll
         for (int s = 0; s < LM_PRE; ++s) {
             const int c0 = (s * 32 + lane) * EPL;
@@ -532,11 +532,11 @@ __global__ void __launch_bounds__(LM_THREADS) k_latent_merge(LatentDecodeArgs a,
     __syncthreads();
     m = sink;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) m = fmaxf(m, red[i]);
+    for (int i = 0; i < LM_WARPS; ++i) m = fmaxf(m, red[i]);
     __syncthreads();
     const float e = exp2f(mine.x - m);
     if (tid < active) ws[tid] = e;
-    const float inv = 1.0f / (cta_sum<8>(e * mine.y, red) + exp2f(sink - m));
+    const float inv = 1.0f / (cta_sum<LM_WARPS>(e * mine.y, red) + exp2f(sink - m));
     for (int x = tid; x < groups * cols; x += LM_THREADS) {
         const int g = x / cols, c = (x % cols) * 4;
         const float* p = a.parts + hs * a.rank + c;
@@ -565,7 +565,7 @@ __global__ void __launch_bounds__(LM_THREADS) k_latent_merge(LatentDecodeArgs a,
         __syncthreads();
     }
 #pragma unroll
-    for (int x = 0; x < LM_ROWS / 8; ++x) {
+    for (int x = 0; x < LM_ROWS / LM_WARPS; ++x) {
         const int r = r0 + x;
         if (r >= a.vdim) break;
         float s = 0.f;
