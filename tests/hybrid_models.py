@@ -41,6 +41,7 @@ MODELS = {
     "no loop, other layers": config([lightning(7, 48, 8), latent(17, 8, 2, 8, 24, base=90.0), (lightning(1, 80, 112), 40), latent(1, 112, 64, 128, 256)],
                                     width=72, vocab=509, mult=1.0, embed_scale=1.0),
     "one pass": config([latent(3, 128, 16, 72, 32), lightning(2, 136, 24)], width=64, vocab=1000, loop=loop(0, 1, 1), mult=0.2),
+    "wide feed-forward": config([(lightning(2, 16, 16), 8160), (latent(1, 16, 4, 16, 24), 12000), (lightning(2, 16, 16), 9000)], width=32, vocab=130),
     "large heads": config([latent(2, 136, 72, 136, 520), lightning(2, 264, 20)], width=80, loop=None),
 }
 
