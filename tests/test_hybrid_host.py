@@ -75,6 +75,21 @@ def test_weights_are_read_and_checked(tmp_path):
         load_hybrid_weights(str(tmp_path))
 
 
+def test_generate_command_line(capsys, tmp_path):
+    from megaqwen_b200 import generate
+    assert generate.main(["--list"]) == 0
+    assert "Satosun: bfloat16, float32" in capsys.readouterr().out
+    with pytest.raises(SystemExit):
+        generate.main([str(tmp_path)])                       # neither ids nor text
+    with pytest.raises(SystemExit):
+        generate.main([str(tmp_path), "--ids", "1", "--prompt", "x"])
+
+
+def test_dtype_is_checked_before_anything_is_built():
+    with pytest.raises(ValueError, match="runs in bfloat16"):
+        registry.build_decoder(weights={"spec": None}, dtype="float32")
+
+
 # ---------------------------------------------------------------- packing
 def test_padding_keeps_products():
     from megaqwen_b200.hybrid import _pad_cols, _pad_rows, _segment

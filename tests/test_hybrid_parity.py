@@ -375,6 +375,18 @@ def test_causal_attention_rejects_what_it_does_not_hold(lib):
     assert call(_lib.MQH_BF16, 20, 16, 16, 0) == -1
 
 
+def test_generate_command(tmp_path):
+    cfg = hm.MODELS["mixed"]
+    w = hm.weights(cfg)
+    hm.save_checkpoint(cfg, w, tmp_path)
+    prompt = hm.tokens(cfg, 21, 10)
+    tokens, margins = ref.HybridReference(cfg, w["tensors"]).greedy(prompt, 12)
+    res = subprocess.run([sys.executable, "-m", "megaqwen_b200.generate", str(tmp_path), "--ids", ",".join(map(str, prompt)), "--max-new", "12",
+                          "--max-seq-len", "64", "--dtype", "float32"], cwd=ROOT, capture_output=True, text=True, timeout=300)
+    assert res.returncode == 0, res.stderr[-2000:]
+    same_tokens([int(t) for t in res.stdout.split()], tokens, margins, 1e-4)
+
+
 # ---------------------------------------------------------------- trace runner
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_trace_run_program(dtype, tmp_path):
