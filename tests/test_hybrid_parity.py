@@ -93,6 +93,45 @@ def test_prompt_portions_and_decoding(name, dtype):
         check(feed(dec, ids, portions), want, dtype, f"{name} {portions[:6]}")
 
 
+ALONE = {
+    "lightning": ([(hm.lightning(3, 48, 32), None)], None, 3.0),
+    "latent attention": ([(hm.latent(3, 48, 20, 32, 72, scale=0.3), None)], None, 3.0),
+    "one head, one pair": ([(hm.latent(1, 16, 2, 16, 16, base=2.0, scale=0.5), None)], None, 3.0),
+    "feed-forward beside it": ([(hm.lightning(1, 16, 16), 176)], None, 3.0),
+    # weights below 1: every pass sends the roundings of the pass before through another norm
+    "loop": ([(hm.lightning(2, 32, 48), None)], hm.loop(0, 1, 4), 0.5),
+    "loop in the middle": ([(hm.lightning(2, 32, 48), None)] * 3, hm.loop(1, 2, 2), 0.5),
+}
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", list(ALONE))
+def test_each_mechanism_alone(name, dtype):
+    """One mechanism per model, added at a weight that lets it carry the logits."""
+    layers, lp, mult = ALONE[name]
+    cfg, oracle, dec = model(hm.config(layers, width=80, vocab=211, loop=lp, mult=mult, embed_scale=0.5), dtype)
+    ids = hm.tokens(cfg, 140, 11)
+    want = oracle_logits(cfg, oracle, ids)
+    for portions in ([140], [], [2, 63, 2, 66]):
+        dec.reset()
+        check(feed(dec, ids, portions), want, dtype, f"{name} {portions}")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("sink", [-30.0, 0.0, 3.0, 30.0])
+def test_sink_from_negligible_to_everything(sink, dtype):
+    from megaqwen_b200.hybrid import HybridDecoder
+    cfg = hm.config([(hm.latent(2, 32, 16, 48, 40, scale=0.3), None)], width=64, vocab=150, mult=3.0, embed_scale=0.5)
+    w = hm.weights(cfg, 12)
+    w["tensors"]["l0.mix.sink"] = torch.tensor([sink, sink / 2]).bfloat16()
+    ids = hm.tokens(cfg, 70, 12)
+    want = ref.HybridReference(cfg, w["tensors"]).forward(ids)
+    dec = HybridDecoder(w, 80, 80, dtype=dtype)
+    for portions in ([70], [3], [2, 40]):
+        dec.reset()
+        check(feed(dec, ids, portions), want, dtype, f"sink {sink} {portions}")
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_long_sequence_over_tile_and_chunk_edges(dtype):
     """Positions around 64-key splits, 128-key tiles and 128-token chunks, in prompts and decoded."""
