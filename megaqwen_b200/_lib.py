@@ -112,18 +112,21 @@ SIGNATURES = {
 
 # ---------------------------------------------------------------- include/megaqwen_hybrid.h
 MQH_BF16, MQH_F32 = 0, 1
-MQH_LIGHTNING, MQH_LATENT = 0, 1
+MQH_LIGHTNING, MQH_LATENT, MQH_GLA, MQH_MAMBA2, MQH_ATTENTION = range(5)
+MQH_PARALLEL, MQH_POST_NORM = 0, 1
 MQH_CHUNK = 128
 MQH_SEGMENT = 32
 
 
 class MqhLayer(C.Structure):
-    _fields_ = [(n, C.c_int) for n in ("kind", "heads", "dim", "vdim", "rank", "rot", "ff", "mix_norm_n")] + [("scale", C.c_float)] + [
-        (n, C.c_void_p) for n in ("norm", "w_in", "w_out", "mix_norm", "decay_pow", "w_ukv", "w_uk_t", "sink", "rope")]
+    _fields_ = [(n, C.c_int) for n in ("kind", "heads", "dim", "vdim", "kv_heads", "rank", "rot", "ff", "mix_norm_n", "norm_parts", "vdim_n", "conv",
+                                       "chunk")] + [(n, C.c_float) for n in ("scale", "inv_tau")] + [
+        (n, C.c_void_p) for n in ("norm", "norm2", "w_in", "w_out", "w_gu", "w_down", "mix_norm", "decay_pow", "w_ukv", "w_uk_t", "sink", "rope", "gate_w",
+                                  "gate_b", "conv_w", "conv_b", "dt_bias", "a_neg", "skip", "q_bias", "k_bias", "q_norm", "k_norm")]
 
 
 class MqhModel(C.Structure):
-    _fields_ = [(n, C.c_int) for n in ("dtype", "width", "norm_n", "vocab", "max_seq")] + [
+    _fields_ = [(n, C.c_int) for n in ("dtype", "form", "width", "norm_n", "vocab", "max_seq")] + [
         (n, C.c_float) for n in ("embed_scale", "eps", "residual_mult")] + [
         (n, C.c_int) for n in ("num_layers", "loop_start", "loop_stop", "loop_times")] + [("layers", C.POINTER(MqhLayer))] + [
         (n, C.c_void_p) for n in ("w_loop", "embed", "final_norm", "head")]
@@ -140,7 +143,7 @@ HYBRID_SIGNATURES = {
     "mqh_run_layer": (C.c_int, [_MODEL, C.c_int]),
     "mqh_state_bytes": (C.c_size_t, [_MODEL, C.c_int]),
     "mqh_state_recurrent": (C.c_int, [_MODEL, C.c_int]),
-    "mqh_in_rows": (C.c_int, [C.POINTER(MqhLayer)]),
+    "mqh_in_rows": (C.c_int, [C.POINTER(MqhLayer), C.c_int]),
     "mqh_ukv_rows": (C.c_int, [C.POINTER(MqhLayer)]),
     "mqh_workspace_bytes": (C.c_size_t, [_MODEL, C.c_int]),
     "mqh_logits_ld": (C.c_int, [_MODEL]),
@@ -148,9 +151,12 @@ HYBRID_SIGNATURES = {
     "mqh_launch_decode": (C.c_int, [_MODEL, _BUF] + [C.c_void_p] * 4 + [C.c_int, C.c_void_p]),
     "mqh_launch_prefill": (C.c_int, [_MODEL, _BUF, C.c_void_p, C.c_int, C.c_int, C.c_void_p, C.c_int, C.c_void_p, C.c_void_p,
                                      C.POINTER(C.c_int), C.c_void_p]),
-    "mqh_lightning_scratch_bytes": (C.c_size_t, [C.c_int] * 4),
+    "mqh_recurrence_scratch_bytes": (C.c_size_t, [C.c_int] * 4),
     "mqh_launch_lightning": (C.c_int, [C.c_int] + [C.c_void_p] * 6 + [C.c_int] * 5 + [C.c_void_p] * 2),
-    "mqh_launch_causal_attention": (C.c_int, [C.c_int] + [C.c_void_p] * 4 + [C.c_int] + [C.c_void_p] * 3 + [C.c_int] * 6 +
+    "mqh_launch_recurrence": (C.c_int, [C.c_int, C.POINTER(MqhLayer)] + [C.c_void_p] * 4 + [C.c_int] + [C.c_void_p] * 2 + [C.c_int] * 2 +
+                              [C.c_void_p] * 2),
+    "mqh_launch_conv": (C.c_int, [C.c_int] + [C.c_void_p] * 5 + [C.c_int] * 4 + [C.c_void_p]),
+    "mqh_launch_causal_attention": (C.c_int, [C.c_int] + [C.c_void_p] * 4 + [C.c_int] + [C.c_void_p] * 4 + [C.c_int] * 8 +
                                     [C.c_float, C.c_int, C.c_void_p, C.c_void_p]),
     "mq_launch_fill_iota": SIGNATURES["mq_launch_fill_iota"],
     "mq_launch_find_first_eos": SIGNATURES["mq_launch_find_first_eos"],

@@ -20,7 +20,7 @@ PKG = os.path.dirname(HERE)
 LIBRARIES = {
     "qwen3": (["decode.cu", "decode_stream.cu", "prefill.cu", "ops.cu", "token_ops.cu"],
               os.environ.get("MQ_LIB_OUT") or os.path.join(PKG, "libmegaqwen_b200.so")),
-    "hybrid": (["hy_linear.cu", "hy_gemv.cu", "hy_rows.cu", "hy_lightning.cu", "hy_latent.cu", "hy_model.cu", "token_ops.cu"],
+    "hybrid": (["hy_linear.cu", "hy_gemv.cu", "hy_rows.cu", "hy_recurrence.cu", "hy_latent.cu", "hy_attention.cu", "hy_model.cu", "token_ops.cu"],
                os.path.join(PKG, "libmegaqwen_hybrid.so")),
 }
 

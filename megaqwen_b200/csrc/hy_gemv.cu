@@ -12,8 +12,9 @@
 // unpacking alone would bound the kernel.
 // 32-bit (k_gemv_f32): a warp per row, FMAs.
 //
-// What the vector is made of (norm of the residual stream, the loop's input, the gated norm of
-// lightning attention beside the feed-forward's activations) is computed by every CTA for itself;
+// What the vector is made of (norm of the residual stream, the loop's input, the gated norm of a
+// recurrence's output beside the feed-forward's activations, the residual stream after the normed
+// result of the sublayer before) is computed by every CTA for itself;
 // what becomes of the result (segments with activations, residual add, LM head with arg-max) is
 // decided row by row at the end.
 #include "hy_common.cuh"
@@ -40,21 +41,89 @@ __device__ __forceinline__ unsigned long long best_key(float v, int i) {
 // latencies, so everything that can be asked for at once is: norm weights before the wait (`Ahead`), the activations
 // that are taken as they are by asynchronous copies, the others in batches of registers.
 constexpr int GV_AHEAD = 2;       // norm weights of the first 2 x 1024 elements
-struct Ahead { float4 gain[GV_AHEAD]; };
+struct Ahead { float4 gain[GV_AHEAD], post[GV_AHEAD]; };
 template <int VEC>
 __device__ __forceinline__ void fetch_gain(const GemvArgs& a, Ahead& h) {
-    const int n = VEC == VEC_NORM ? a.K : VEC == VEC_GATED ? a.hv : 0;
+    const float* w = VEC == VEC_GATED ? a.gn.w : a.gain;
+    const int n = VEC == VEC_NORM || VEC == VEC_POST_NORM ? a.K : VEC == VEC_GATED ? a.gn.hv : 0;
+    const int np = (VEC == VEC_POST || VEC == VEC_POST_NORM) && a.post_y ? a.K : 0;
 #pragma unroll
     for (int x = 0; x < GV_AHEAD; ++x) {
         const int i = (threadIdx.x + x * GV_THREADS) * 4;
-        h.gain[x] = i < n ? load4(a.gain + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        h.gain[x] = i < n ? load4(w + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        h.post[x] = i < np ? load4(a.post + i) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
 }
+__device__ __forceinline__ float sum_sq(const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
 template <typename T, int VEC>
-__device__ __forceinline__ void make_vector(const GemvArgs& a, const Ahead& ahead, T* vec, float* raw, float* red) {
+__device__ __forceinline__ void make_vector(const GemvArgs& a, const Ahead& ahead, T* vec, float* raw, float* scratch, float* red) {
     const int tid = threadIdx.x, K = a.K;
     constexpr int STRIDE = GV_THREADS * 4;
-    if (VEC == VEC_NORM || VEC == VEC_CONCAT) {
+    if (VEC == VEC_POST || VEC == VEC_POST_NORM) {
+        const T* erow = nullptr;
+        if (a.token) {
+            int tok = *a.token;
+            if (tok < 0 || tok >= a.vocab) {
+                if (tid == 0) atomicOr(a.status, MQ_STATUS_BAD_TOKEN);
+                tok = tok < 0 ? 0 : a.vocab - 1;
+            }
+            erow = reinterpret_cast<const T*>(a.embed) + (size_t)tok * K;
+        }
+        auto stream = [&](int i) {
+            if (!erow) return load4_cg(a.x + i);
+            const float4 v = load4(erow + i);
+            return make_float4(v.x * a.embed_scale, v.y * a.embed_scale, v.z * a.embed_scale, v.w * a.embed_scale);
+        };
+        // the first quads stay in registers, further ones of the result wait in shared memory
+        float4 xk[GV_AHEAD], yk[GV_AHEAD];
+        float ss = 0.f, inv = 0.f;
+#pragma unroll
+        for (int x = 0; x < GV_AHEAD; ++x) {
+            const int i = tid * 4 + x * STRIDE;
+            xk[x] = yk[x] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < K) {
+                xk[x] = stream(i);
+                if (a.post_y) yk[x] = load4_cg(a.post_y + i);
+            }
+        }
+        if (a.post_y) {
+#pragma unroll
+            for (int x = 0; x < GV_AHEAD; ++x) ss += sum_sq(yk[x]);
+            for (int i = tid * 4 + GV_AHEAD * STRIDE; i < K; i += STRIDE) {
+                const float4 y = load4_cg(a.post_y + i);
+                ss += sum_sq(y);
+                store4(raw + i, y);
+            }
+            inv = 1.0f / sqrtf(cta_sum<GV_WARPS>(ss, red) / (float)a.norm_n + a.eps);
+        }
+        ss = 0.f;
+        auto put = [&](int i, float4 v, const float4& y, const float4& g) {
+            if (a.post_y) {
+                v.x = fmaf(y.x * inv, g.x, v.x); v.y = fmaf(y.y * inv, g.y, v.y);
+                v.z = fmaf(y.z * inv, g.z, v.z); v.w = fmaf(y.w * inv, g.w, v.w);
+            }
+            if (blockIdx.x == 0 && a.x_store) store4(a.x_store + i, v);
+            if (VEC == VEC_POST_NORM) { ss += sum_sq(v); store4(raw + i, v); }
+            else store4(vec + i, v);
+        };
+#pragma unroll
+        for (int x = 0; x < GV_AHEAD; ++x) {
+            const int i = tid * 4 + x * STRIDE;
+            if (i < K) put(i, xk[x], yk[x], ahead.post[x]);
+        }
+        for (int i = tid * 4 + GV_AHEAD * STRIDE; i < K; i += STRIDE) {
+            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+            put(i, stream(i), a.post_y ? load4(raw + i) : zero, a.post_y ? load4(a.post + i) : zero);
+        }
+        if (VEC == VEC_POST_NORM) {
+            inv = 1.0f / sqrtf(cta_sum<GV_WARPS>(ss, red) / (float)a.norm_n + a.eps);
+            int n = 0;
+            for (int i = tid * 4; i < K; i += STRIDE, ++n) {
+                const float4 v = load4(raw + i), g = n == 0 ? ahead.gain[0] : n == 1 ? ahead.gain[1] : load4(a.gain + i);
+                store4(vec + i, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
+            }
+        }
+    } else if (VEC == VEC_NORM || VEC == VEC_CONCAT) {
         const int width = VEC == VEC_CONCAT ? K / 2 : K;
         const T* erow = nullptr;
         if (a.token) {
@@ -104,40 +173,12 @@ __device__ __forceinline__ void make_vector(const GemvArgs& a, const Ahead& ahea
             }
         }
     } else {
-        const int hv = VEC == VEC_GATED ? a.hv : 0;
+        const int hv = VEC == VEC_GATED ? a.gn.hv : 0;
         const T* cat = reinterpret_cast<const T*>(a.cat);
         constexpr int E = Elem<T>::PER16;
         for (int i = hv + tid * E; i < K; i += GV_THREADS * E) cp_async16(vec + i, cat + i);
         cp_async_commit();
-        if (VEC == VEC_GATED) {
-            const T* gate = reinterpret_cast<const T*>(a.g);
-            float ss = 0.f;
-            int n = 0;
-            for (int i0 = tid * 4; i0 < hv; i0 += 2 * STRIDE, n += 2) {
-                float4 v[2], g[2];
-#pragma unroll
-                for (int x = 0; x < 2; ++x) {
-                    const int i = i0 + x * STRIDE;
-                    if (i >= hv) break;
-                    v[x] = load4_cg(a.o + i);
-                    g[x] = load4_cg(gate + i);
-                }
-#pragma unroll
-                for (int x = 0; x < 2; ++x) {
-                    const int i = i0 + x * STRIDE;
-                    if (i >= hv) break;
-                    const float4 w = n == 0 ? ahead.gain[x] : load4(a.gain + i);
-                    ss += v[x].x * v[x].x + v[x].y * v[x].y + v[x].z * v[x].z + v[x].w * v[x].w;
-                    store4(raw + i, make_float4(v[x].x * w.x * Elem<T>::sigmoid(g[x].x), v[x].y * w.y * Elem<T>::sigmoid(g[x].y),
-                                                v[x].z * w.z * Elem<T>::sigmoid(g[x].z), v[x].w * w.w * Elem<T>::sigmoid(g[x].w)));
-                }
-            }
-            const float inv = 1.0f / sqrtf(cta_sum<GV_WARPS>(ss, red) / (float)a.norm_n + a.eps);
-            for (int i = tid * 4; i < hv; i += STRIDE) {
-                const float4 v = load4(raw + i);
-                store4(vec + i, make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv));
-            }
-        }
+        if (VEC == VEC_GATED) gated_norm_row<T, GV_WARPS>(a.gn, ahead.gain, raw, scratch, red, vec);
         cp_async_wait_all();
     }
 }
@@ -153,6 +194,7 @@ __device__ __forceinline__ void put_rows(const GemvArgs& a, int first, int cnt, 
             const int c = r - s.row0;
             if (c >= s.rows) continue;
             float y0 = value(2 * p), y1 = value(2 * p + 1);
+            if (s.bias) { y0 += s.bias[c]; y1 += s.bias[c + 1]; }
             if (s.act == ACT_SWIGLU) {
                 reinterpret_cast<T*>(s.out)[c / 2] = Elem<T>::put(silu<T>(y0) * y1);
             } else {
@@ -226,7 +268,7 @@ __global__ void __launch_bounds__(GV_THREADS, 2) k_gemv_mma(GemvArgs a) {
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, c8 = (lane & 3) * 8;
     const int K = a.K, nsteps = (K + 31) / 32;
     bf16* xs = reinterpret_cast<bf16*>(gm_raw);                   // [nsteps * 32]
-    float* raw = reinterpret_cast<float*>(xs + nsteps * 32);      // [K] (VEC_NORM, VEC_GATED)
+    float* raw = reinterpret_cast<float*>(xs + nsteps * 32);      // [K] (norms), then what the gated norm needs
     const bf16* W = reinterpret_cast<const bf16*>(a.W);
     int r0, r1;
     my_rows<OUT>(a.rows, r0, r1);
@@ -263,7 +305,7 @@ __global__ void __launch_bounds__(GV_THREADS, 2) k_gemv_mma(GemvArgs a) {
     // may read cache rows and states ahead of its own waits.
     if (OUT == OUT_HEAD) pdl_trigger();
     const float y_ahead = OUT == OUT_ADD && tid < r1 - r0 ? __ldcg(a.y + r0 + tid) : 0.f;
-    make_vector<bf16, VEC>(a, ahead, xs, raw, red);
+    make_vector<bf16, VEC>(a, ahead, xs, raw, raw + K, red);
     if (tid < nsteps * 32 - K) xs[K + tid] = __float2bfloat16_rn(0.f);
     __syncthreads();
 
@@ -338,7 +380,7 @@ __global__ void __launch_bounds__(GV_THREADS, 2) k_gemv_f32(GemvArgs a) {
     if (OUT != OUT_HEAD) pdl_trigger();
     pdl_wait_cta();
     if (OUT == OUT_HEAD) pdl_trigger();
-    make_vector<float, VEC>(a, ahead, gf_vec, gf_vec, red);
+    make_vector<float, VEC>(a, ahead, gf_vec, gf_vec, gf_vec + K, red);
     __syncthreads();
     unsigned long long best = 0ull;
     for (int first = r0 + warp * 2; first < r1; first += GV_WARPS * 2) {      // two rows (a pair) at a time
@@ -362,9 +404,11 @@ __global__ void __launch_bounds__(GV_THREADS, 2) k_gemv_f32(GemvArgs a) {
 }
 
 // ---------------------------------------------------------------- launches
+template <int VEC>
+static size_t vec_scratch(const GemvArgs& a) { return VEC == VEC_GATED ? (size_t)gated_scratch(a.gn) * 4 : 0; }
 template <int VEC, int OUT, bool TALL>
 static int go_mma(Stream& st, const GemvArgs& a) {
-    const size_t smem = (size_t)((a.K + 31) / 32) * 64 + (VEC == VEC_NORM || VEC == VEC_GATED ? (size_t)a.K * 4 : 0);
+    const size_t smem = (size_t)((a.K + 31) / 32) * 64 + (VEC == VEC_CONCAT || VEC == VEC_PLAIN ? 0 : (size_t)a.K * 4) + vec_scratch<VEC>(a);
     const int rc = allow_smem(k_gemv_mma<VEC, OUT, TALL>, smem);
     if (rc) return rc;
     // The LM head is long enough to fill the device by itself: two CTAs per SM keep more loads in flight.  The products of
@@ -378,9 +422,10 @@ static int go(Stream& st, const GemvArgs& a, const bf16*) {
 }
 template <int VEC, int OUT>
 static int go(Stream& st, const GemvArgs& a, const float*) {
-    const int rc = allow_smem(k_gemv_f32<VEC, OUT>, (size_t)a.K * 4);
+    const size_t smem = (size_t)a.K * 4 + vec_scratch<VEC>(a);
+    const int rc = allow_smem(k_gemv_f32<VEC, OUT>, smem);
     if (rc) return rc;
-    return launch(st, k_gemv_f32<VEC, OUT>, dim3(sm_count()), dim3(GV_THREADS), (size_t)a.K * 4, a);
+    return launch(st, k_gemv_f32<VEC, OUT>, dim3(sm_count()), dim3(GV_THREADS), smem, a);
 }
 template <typename T>
 int gemv(Stream& st, int vec, int out, const GemvArgs& a) {
@@ -390,6 +435,10 @@ int gemv(Stream& st, int vec, int out, const GemvArgs& a) {
     if (vec == VEC_CONCAT && out == OUT_STORE) return go<VEC_CONCAT, OUT_STORE>(st, a, t);
     if (vec == VEC_GATED && out == OUT_ADD) return go<VEC_GATED, OUT_ADD>(st, a, t);
     if (vec == VEC_PLAIN && out == OUT_ADD) return go<VEC_PLAIN, OUT_ADD>(st, a, t);
+    if (vec == VEC_GATED && out == OUT_STORE) return go<VEC_GATED, OUT_STORE>(st, a, t);
+    if (vec == VEC_PLAIN && out == OUT_STORE) return go<VEC_PLAIN, OUT_STORE>(st, a, t);
+    if (vec == VEC_POST && out == OUT_SEGMENTS) return go<VEC_POST, OUT_SEGMENTS>(st, a, t);
+    if (vec == VEC_POST_NORM && out == OUT_HEAD) return go<VEC_POST_NORM, OUT_HEAD>(st, a, t);
     return MQ_ERR_BAD_ARG;
 }
 template int gemv<bf16>(Stream&, int, int, const GemvArgs&);

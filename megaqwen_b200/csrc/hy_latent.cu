@@ -16,8 +16,6 @@
 namespace mq {
 namespace hy {
 
-constexpr float LOG2E = 1.4426950408889634f;
-
 // The interleaved rotation: elements 2i, 2i + 1 turn by the angle whose cos, sin are rope[i].
 __device__ __forceinline__ float2 rotate_pair(float u, float v, float2 cs) { return make_float2(u * cs.x - v * cs.y, v * cs.x + u * cs.y); }
 __device__ __forceinline__ float2 load2(const float* p) { return __ldcg(reinterpret_cast<const float2*>(p)); }
@@ -106,7 +104,8 @@ int latent_rows(Stream& st, const LatentRowsArgs& a) {
 template int latent_rows<bf16>(Stream&, const LatentRowsArgs&);
 template int latent_rows<float>(Stream&, const LatentRowsArgs&);
 
-// Causal attention without tensor cores: one CTA per (row, head), tiles of 128 keys, online softmax.
+// Causal attention (all keys before a position, or those of its chunk) without tensor cores: one CTA per (row, head), tiles of 128 keys, online
+// softmax.
 constexpr int CR_KEYS = 128, CR_MAXV = 4;
 template <typename T>
 __global__ void __launch_bounds__(128) k_causal_rows(CausalArgs a) {
@@ -116,7 +115,7 @@ __global__ void __launch_bounds__(128) k_causal_rows(CausalArgs a) {
     __shared__ float p[CR_KEYS];
     __shared__ float red[4];
     const int t = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int nk = a.pos0 + t + 1;
+    const int nk = a.pos0 + t + 1, first = a.chunk > 0 ? (nk - 1) / a.chunk * a.chunk : 0, kvh = head / (a.heads / a.kv_heads);
     const T* q = reinterpret_cast<const T*>(a.q) + ((size_t)t * a.heads + head) * a.dim;
     const T* qr = reinterpret_cast<const T*>(a.q_rot) + ((size_t)t * a.heads + head) * a.rot;
     const T* kr = reinterpret_cast<const T*>(a.k_rot);
@@ -127,11 +126,11 @@ __global__ void __launch_bounds__(128) k_causal_rows(CausalArgs a) {
     float m = a.sink ? a.sink[head] * LOG2E : -INFINITY;
     float l = a.sink ? 1.0f : 0.0f;                      // the sink is a key without a value
     float acc[CR_MAXV] = {};
-    for (int k0 = 0; k0 < nk; k0 += CR_KEYS) {
+    for (int k0 = first; k0 < nk; k0 += CR_KEYS) {
         const int cnt = min(CR_KEYS, nk - k0);
         float best = -INFINITY;
         for (int j = warp; j < cnt; j += 4) {
-            const T* k = reinterpret_cast<const T*>(a.k) + ((size_t)(k0 + j) * a.heads + head) * a.dim;
+            const T* k = reinterpret_cast<const T*>(a.k) + (size_t)(k0 + j) * a.ldk + (size_t)kvh * a.dim;
             float s = 0.f;
             for (int i = lane * 4; i < a.dim; i += 128) {
                 const float4 kv = load4(k + i), qv = load4(cr_q + i);
@@ -154,18 +153,19 @@ __global__ void __launch_bounds__(128) k_causal_rows(CausalArgs a) {
         for (int x = 0; x < CR_MAXV; ++x) {
             const int j = tid + x * 128;
             if (j >= a.vdim) break;
-            const T* v = reinterpret_cast<const T*>(a.v) + ((size_t)k0 * a.heads + head) * a.vdim + j;
+            const T* v = reinterpret_cast<const T*>(a.v) + (size_t)k0 * a.ldv + (size_t)kvh * a.vdim + j;
             float s = 0.f;
-            for (int y = 0; y < cnt; ++y) s = fmaf(p[y], Elem<T>::get(v[(size_t)y * a.heads * a.vdim]), s);
+            for (int y = 0; y < cnt; ++y) s = fmaf(p[y], Elem<T>::get(v[(size_t)y * a.ldv]), s);
             acc[x] = acc[x] * alpha + s;
         }
         __syncthreads();
     }
+    const float gate = a.gate ? 1.0f / (1.0f + expf(-a.gate[(size_t)t * a.ld_gate + head])) : 1.0f;
     T* o = reinterpret_cast<T*>(a.out) + (size_t)t * a.ld_out + (size_t)head * a.vdim;
 #pragma unroll
     for (int x = 0; x < CR_MAXV; ++x) {
         const int j = tid + x * 128;
-        if (j < a.vdim) o[j] = Elem<T>::put(acc[x] / l);
+        if (j < a.vdim) o[j] = Elem<T>::put(acc[x] / l * gate);
     }
 }
 template <typename T>
@@ -179,17 +179,25 @@ template int causal_simt<float>(Stream&, const CausalArgs&);
 // The tcgen05 kernel holds heads of up to 128 + 64 query / key and 128 value dimensions, and takes a positive scale.
 bool causal_tc_fits(int dim, int rot, int vdim, float scale) { return dim <= 128 && rot <= 64 && vdim <= 128 && scale > 0.f; }
 int causal_tc(Stream& st, const CausalArgs& a) {
-    const uint64_t n = a.n, keys = a.pos0 + a.n, H = a.heads;
+    const uint64_t n = a.n, keys = a.pos0 + a.n, H = a.heads, G = a.kv_heads;
     CUtensorMap mq_, mk, mv, mqr, mkr;
     int rc = get_map(a.q, n, a.dim, H * a.dim, TA_BQ, &mq_, H, a.dim);
-    if (!rc) rc = get_map(a.q_rot, n, a.rot, H * a.rot, TA_BQ, &mqr, H, a.rot);
-    if (!rc) rc = get_map(a.k, keys, a.dim, H * a.dim, TA_BK, &mk, H, a.dim);
-    if (!rc) rc = get_map(a.k_rot, keys, a.rot, a.ld_rot, TA_BK, &mkr, 1, keys * a.ld_rot);
-    if (!rc) rc = get_map(a.v, keys, a.vdim, H * a.vdim, TA_BK, &mv, H, a.vdim);
+    if (!rc) rc = get_map(a.k, keys, a.dim, a.ldk, TA_BK, &mk, G, a.dim);
+    if (!rc) rc = get_map(a.v, keys, a.vdim, a.ldv, TA_BK, &mv, G, a.vdim);
+    if (!rc && a.rot) rc = get_map(a.q_rot, n, a.rot, H * a.rot, TA_BQ, &mqr, H, a.rot);
+    if (!rc && a.rot) rc = get_map(a.k_rot, keys, a.rot, a.ld_rot, TA_BK, &mkr, 1, keys * a.ld_rot);
     if (rc) return rc;
-    const AttnTcArgs t = {(bf16*)a.out, a.ld_out, a.vdim, a.n, a.pos0, 1, 0, a.dim / 16, a.rot / 16, a.scale * LOG2E, a.sink, a.status};
+    AttnTcArgs t = {(bf16*)a.out, a.ld_out, a.vdim, a.n, a.pos0, a.heads / a.kv_heads, 0, a.dim / 16, a.rot / 16, a.scale * LOG2E, a.sink, a.status};
+    t.chunk = a.chunk; t.gate = a.gate; t.ld_gate = a.ld_gate;
     ++st.launches;
     const int qp = (a.dim + 63) / 64, vp = (a.vdim + 63) / 64;
+    if (a.rot == 0) {                  // no shared key part
+        if (qp == 1 && vp == 1) return launch_attention_tc<1, 0, 1>(a.heads, mq_, mk, mv, mq_, mk, t, st.s);
+        if (qp == 1 && vp == 2) return launch_attention_tc<1, 0, 2>(a.heads, mq_, mk, mv, mq_, mk, t, st.s);
+        if (qp == 2 && vp == 1) return launch_attention_tc<2, 0, 1>(a.heads, mq_, mk, mv, mq_, mk, t, st.s);
+        if (qp == 2 && vp == 2) return launch_attention_tc<2, 0, 2>(a.heads, mq_, mk, mv, mq_, mk, t, st.s);
+        return MQ_ERR_UNSUPPORTED;
+    }
     if (qp == 1 && vp == 1) return launch_attention_tc<1, 1, 1>(a.heads, mq_, mk, mv, mqr, mkr, t, st.s);
     if (qp == 1 && vp == 2) return launch_attention_tc<1, 1, 2>(a.heads, mq_, mk, mv, mqr, mkr, t, st.s);
     if (qp == 2 && vp == 1) return launch_attention_tc<2, 1, 1>(a.heads, mq_, mk, mv, mqr, mkr, t, st.s);

@@ -47,6 +47,9 @@ struct AttnTcArgs {
     float c;                 // score scale * log2(e), positive
     const float* sink;       // per head: the denominator also holds exp(sink); null for none
     unsigned int* status;
+    int chunk = 0;           // > 0: position i sees keys from i / chunk * chunk on, else from 0
+    const float* gate = nullptr;   // [S, ld_gate] per row and head: the output is multiplied by sigmoid(gate); null for none
+    int ld_gate = 0;
 };
 
 
@@ -84,7 +87,8 @@ k_attention_tc(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
     const int head = blockIdx.x, plane = a.kv_plane0 + head / a.kv_group;
     const int q0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * TA_BQ;        // longest query tiles first
     const int kv_end = min(pos0 + S, pos0 + q0 + TA_BQ);                  // keys any row of the tile may see
-    const int nt = (kv_end + TA_BK - 1) / TA_BK;
+    const int kbase = a.chunk > 0 ? (pos0 + q0) / a.chunk * a.chunk : 0;  // first key of the tile's first row: key tiles start here
+    const int nt = (kv_end - kbase + TA_BK - 1) / TA_BK;
 
     if (tid == 0) {
         mbar_init(q_full, 1);
@@ -114,13 +118,13 @@ k_attention_tc(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
                 if (j >= 2 && !mbar_wait(&k_empty[st], (uint32_t)((j >> 1) - 1) & 1u, status)) break;
                 mbar_expect_tx(&k_full[st], Cfg::Q_BYTES);
 #pragma unroll
-                for (int p = 0; p < QP; ++p) tma_load_3d(sK + st * Cfg::Q_BYTES + p * TA_PANEL_BYTES, &tmK, p * 64, j * TA_BK, plane, &k_full[st]);
+                for (int p = 0; p < QP; ++p) tma_load_3d(sK + st * Cfg::Q_BYTES + p * TA_PANEL_BYTES, &tmK, p * 64, kbase + j * TA_BK, plane, &k_full[st]);
 #pragma unroll
-                for (int p = 0; p < RP; ++p) tma_load_3d(sK + st * Cfg::Q_BYTES + (QP + p) * TA_PANEL_BYTES, &tmKr, p * 64, j * TA_BK, 0, &k_full[st]);
+                for (int p = 0; p < RP; ++p) tma_load_3d(sK + st * Cfg::Q_BYTES + (QP + p) * TA_PANEL_BYTES, &tmKr, p * 64, kbase + j * TA_BK, 0, &k_full[st]);
                 if (j >= 2 && !mbar_wait(&v_empty[st], (uint32_t)((j >> 1) - 1) & 1u, status)) break;
                 mbar_expect_tx(&v_full[st], Cfg::V_BYTES);
 #pragma unroll
-                for (int p = 0; p < VP; ++p) tma_load_3d(sV + st * Cfg::V_BYTES + p * TA_PANEL_BYTES, &tmV, p * 64, j * TA_BK, plane, &v_full[st]);
+                for (int p = 0; p < VP; ++p) tma_load_3d(sV + st * Cfg::V_BYTES + p * TA_PANEL_BYTES, &tmV, p * 64, kbase + j * TA_BK, plane, &v_full[st]);
             }
         }
         __syncwarp();
@@ -189,6 +193,7 @@ k_attention_tc(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
         const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
         const uint32_t col_off = (uint32_t)(half * 64), out_off = (uint32_t)(half * OC);
         const int qpos = pos0 + q0 + r;                       // absolute position of this thread's query
+        const int qfirst = a.chunk > 0 ? qpos / a.chunk * a.chunk : 0;
         const float c = a.c;
         float m = -INFINITY, l = 0.f;                         // m: the maximum the sums are scaled to (raw score units)
         bool ok = true;
@@ -198,8 +203,8 @@ k_attention_tc(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
             const uint32_t ts = tmem_base + st * 128 + lane_off + col_off;
             ok = ok && mbar_wait(&s_full[st], (uint32_t)(j >> 1) & 1u, status);
             tc_fence_after();
-            const int k0 = j * TA_BK + half * 64;             // first key of this thread's half
-            const bool diag = k0 + 63 > qpos;                 // some keys of this half lie beyond the query
+            const int k0 = kbase + j * TA_BK + half * 64;     // first key of this thread's half
+            const bool diag = k0 + 63 > qpos || k0 < qfirst;  // some keys of this half lie beyond the query, or before its chunk
             uint32_t sv[64];
 #pragma unroll
             for (int cb = 0; cb < 2; ++cb) tmem_ld32_nowait(ts + cb * 32, *reinterpret_cast<uint32_t(*)[32]>(&sv[cb * 32]));
@@ -207,10 +212,10 @@ k_attention_tc(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
             tc_fence_before();
             mbar_arrive(&s_free[st]);                         // the scores are in registers: S[st] may be overwritten
             float mh = -INFINITY;
-            if (__any_sync(0xffffffffu, diag)) {              // only the last one or two key tiles of a query tile
+            if (__any_sync(0xffffffffu, diag)) {              // without chunks only the last one or two key tiles of a query tile
 #pragma unroll
                 for (int i = 0; i < 64; ++i) {
-                    if (k0 + i > qpos) sv[i] = 0xff800000u;   // -inf
+                    if (k0 + i > qpos || k0 + i < qfirst) sv[i] = 0xff800000u;   // -inf
                     mh = fmaxf(mh, __uint_as_float(sv[i]));
                 }
             } else {
@@ -249,7 +254,8 @@ k_attention_tc(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
                 l *= alpha;
                 if (grow) m = mx;
             }
-            const float mc = m * c;
+            // a row whose chunk begins in a later key tile has seen nothing yet: all its weights are 0
+            const float mc = m == -INFINITY ? 0.f : m * c;
             // (S[st] last held the probabilities of tile j - 2; their product was issued before the Q K^T of this tile)
             // probabilities -> bf16 pairs -> A operand of the P V product in tensor memory; this thread's 64 keys
             // are 32 packed columns
@@ -277,7 +283,8 @@ k_attention_tc(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
         pair_sync();
         float den = xm[r][0] + xm[r][1];
         if (a.sink) den += fast_exp2(fmaf(a.sink[head], 1.4426950408889634f, -m * c));   // no value, and not scaled
-        const float inv = 1.0f / den;
+        float inv = 1.0f / den;
+        if (a.gate && q0 + r < S) inv *= 1.0f / (1.0f + __expf(-a.gate[(size_t)(q0 + r) * a.ld_gate + head]));
         bf16* orow = a.out + (size_t)(q0 + r) * a.ld_out + head * a.head_cols + half * OC;
         const int cols = a.head_cols - half * OC;             // value columns left for this thread
 #pragma unroll

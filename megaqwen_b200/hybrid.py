@@ -1,7 +1,8 @@
-"""Decoder of layer-listed models (design "Satosun"): each layer has its own
-mixer (lightning attention or latent attention) beside an optional gated
+"""Decoder of layer-listed models: each layer has its own mixer and an optional
+gated feed-forward.  Design "Satosun": lightning or latent attention beside the
 feed-forward, and a stretch of layers may run several times with the same
-weights.
+weights.  Design "Vunasun": gated linear attention, Mamba-2 or chunked attention,
+the feed-forward after it, norms on their results.
 
 The object has the interface of ``MegakernelDecoder`` (engine.py): prompts,
 portions of prompts, single steps, device-resident chains replayed from CUDA
@@ -58,12 +59,12 @@ def decay_powers(decay, count: int) -> torch.Tensor:
     return (d[:, None] ** torch.arange(count, dtype=torch.float64)[None, :]).to(torch.float32)
 
 
-def interleaved_rope_table(max_seq_len: int, dims: int, base: float) -> torch.Tensor:
-    """[max_seq_len, pad16(dims)/2, 2] fp32: cos, sin of position * base^(-2i/dims) for the pair (2i, 2i + 1);
-    the pairs of the padding do not turn."""
+def rope_table(max_seq_len: int, dims: int, base: float, padded: int | None = None) -> torch.Tensor:
+    """[max_seq_len, padded/2, 2] fp32: cos, sin of position * base^(-2i/dims) for pair i, (2i, 2i + 1) or
+    (i, i + dims/2); pairs of the padding do not turn."""
     f = base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
     a = torch.arange(max_seq_len, dtype=torch.float64)[:, None] * f[None, :]
-    a = torch.nn.functional.pad(a, (0, (pad16(dims) - dims) // 2))
+    a = torch.nn.functional.pad(a, (0, ((padded or dims) - dims) // 2))
     return torch.stack([torch.cos(a), torch.sin(a)], -1).to(torch.float32).contiguous()
 
 
@@ -97,7 +98,7 @@ class HybridDecoder(DecodeEngine):
             nbytes = lib.mqh_workspace_bytes(C.byref(self._model), self.max_prefill_len_)
             if nbytes == 0:
                 raise RuntimeError("this model has sizes that the kernels do not hold "
-                                   "(lightning dim <= 512, latent rank <= 2048, latent vdim <= 512)")
+                                   "(a head's query / key or state size <= 512, latent rank <= 2048, latent vdim <= 512, convolution <= 64 taps)")
             self._workspace = torch.zeros(nbytes, dtype=torch.uint8, device=device)
             self._buf = MqhBuffers(_ptr(self._workspace), nbytes, self.max_prefill_len_, self.state.pointers, _ptr(self._scalars) + 4)
             self._step_launches = lib.mqh_decode_launch_count(C.byref(self._model))
@@ -123,30 +124,38 @@ class HybridDecoder(DecodeEngine):
 
         w = spec.hidden_size
 
-        def gain(name):                      # norms over the width are stored around zero
-            return self._keep(_pad_vec(1.0 + vec(name), 1, w) * _pad_vec(torch.ones(w, device=dev), 1, w))
+        def gain(name, scale=None):          # norms over the width: stored around zero, or plain with a layer scale
+            g = 1.0 + vec(name) if not spec.post_norm else vec(name) * (vec(scale) if scale else 1.0)
+            return self._keep(_pad_vec(g, 1, w))
 
+        pack = {"lightning": self._pack_lightning, "latent_attention": self._pack_latent, "gla": self._pack_gla, "mamba2": self._pack_mamba2,
+                "attention": self._pack_attention}
+        form = _lib.MQH_POST_NORM if spec.post_norm else _lib.MQH_PARALLEL
         self._layers = (MqhLayer * spec.num_layers)()
         for i, layer in enumerate(spec.layers):
             p, m, out = f"l{i}.", layer.mixer, self._layers[i]
             out.heads, out.dim, out.vdim, out.ff = m.heads, pad16(m.dim), pad16(m.vdim), pad16(layer.ff)
-            out.norm = gain(p + "norm1")
-            pack = self._pack_lightning if m.kind == "lightning" else self._pack_latent
-            rows = pack(out, m, p + "mix.", mat, vec)
+            out.vdim_n, out.norm_parts = m.vdim, 1
+            out.norm = gain(p + "norm1", p + "ls1")
+            rows = pack[m.kind](out, m, p + "mix.", mat, vec)
             cols = [_pad_cols(mat(p + "mix.o"), m.heads, m.vdim)]
             if layer.ff:
                 gate, up = (_pad_rows(mat(p + "mlp." + n), 1, layer.ff) for n in ("gate", "up"))
-                rows.append(torch.stack([gate, up], 1).reshape(2 * gate.shape[0], -1))
-                cols.append(_pad_cols(mat(p + "mlp.down"), 1, layer.ff))
+                gu, down = torch.stack([gate, up], 1).reshape(2 * gate.shape[0], -1), _pad_cols(mat(p + "mlp.down"), 1, layer.ff)
+                if spec.post_norm:
+                    out.w_gu, out.w_down, out.norm2 = self._keep(_segment(gu)), self._keep(down), gain(p + "norm2", p + "ls2")
+                else:
+                    rows.append(gu)
+                    cols.append(down)
             w_in = torch.cat([_segment(r) for r in rows])
-            if w_in.shape[0] != self._lib.mqh_in_rows(C.byref(out)):
+            if w_in.shape[0] != self._lib.mqh_in_rows(C.byref(out), form):
                 raise RuntimeError("packed input projection does not have the rows the library expects")
             out.w_in = self._keep(w_in)
             out.w_out = self._keep(torch.cat(cols, 1))
         wp = pad16(w)
         loop = spec.loop or (0, 0, 0)
         self._model = MqhModel(
-            code, wp, w, spec.vocab_size, self.max_seq_len_, spec.embed_scale, spec.rms_eps, spec.residual_mult, spec.num_layers, *loop,
+            code, form, wp, w, spec.vocab_size, self.max_seq_len_, spec.embed_scale, spec.rms_eps, spec.residual_mult, spec.num_layers, *loop,
             self._layers, self._keep(_pad_cols(mat("loop.in"), 2, w)) if spec.loop else None,
             self._keep(torch.nn.functional.pad(mat("embed"), (0, wp - w))), gain("final.norm"),
             self._keep(torch.nn.functional.pad(mat("head"), (0, wp - w))))
@@ -157,14 +166,49 @@ class HybridDecoder(DecodeEngine):
         out.decay_pow = self._keep(decay_powers(m.decay, _lib.MQH_CHUNK + 1).to(self.device))
         return [_pad_rows(mat(p + n), m.heads, d) for n, d in (("q", m.dim), ("k", m.dim), ("v", m.vdim), ("g", m.vdim))]
 
+    def _rope(self, dims: int, base: float, padded: int) -> int:
+        key = (dims, base, padded)
+        if key not in self._ropes:
+            self._ropes[key] = self._keep(rope_table(self.max_seq_len_, dims, base, padded).to(self.device))
+        return self._ropes[key]
+
+    def _pack_gla(self, out: MqhLayer, m: MixerSpec, p: str, mat, vec) -> list:
+        out.kind, out.rank, out.scale, out.inv_tau = _lib.MQH_GLA, pad16(m.rank), m.dim ** -0.5, 1.0 / m.tau
+        out.mix_norm_n, out.norm_parts = m.vdim, m.heads                     # every head by itself, one weight for all
+        out.mix_norm = self._keep(_pad_vec(vec(p + "norm").repeat(m.heads), m.heads, m.vdim))
+        a2 = _pad_rows(mat(p + "a2"), m.heads, m.dim)
+        out.gate_w = self._keep(a2.reshape(m.heads, pad16(m.dim), pad16(m.rank)).transpose(1, 2))
+        out.gate_b = self._keep(_pad_vec(vec(p + "a2.b"), m.heads, m.dim))
+        return [_pad_rows(mat(p + n), h, d) for n, h, d in
+                (("q", m.heads, m.dim), ("k", m.heads, m.dim), ("v", m.heads, m.vdim), ("g", m.heads, m.vdim), ("a1", 1, m.rank))]
+
+    def _pack_mamba2(self, out: MqhLayer, m: MixerSpec, p: str, mat, vec) -> list:
+        out.kind, out.kv_heads, out.conv = _lib.MQH_MAMBA2, m.kv_heads, m.conv
+        out.mix_norm_n, out.norm_parts = m.heads * m.vdim // m.norm_groups, m.norm_groups
+        out.mix_norm = self._keep(_pad_vec(vec(p + "norm"), m.heads, m.vdim))
+        out.dt_bias, out.skip = self._keep(vec(p + "dt_bias")), self._keep(vec(p + "D"))
+        out.a_neg = self._keep((-torch.exp(vec(p + "A_log").double())).float())
+        inner, gn = m.heads * m.vdim, m.kv_heads * m.dim
+        parts = ((inner, m.heads, m.vdim), (gn, m.kv_heads, m.dim), (gn, m.kv_heads, m.dim))           # x, B, C
+        sizes = [n for n, _, _ in parts]
+        conv = [_pad_rows(c, h, d) for c, (_, h, d) in zip(vec(p + "conv").split(sizes), parts)]
+        out.conv_w = self._keep(torch.cat(conv)[:, :m.conv].T)
+        out.conv_b = self._keep(torch.cat([_pad_vec(c, h, d) for c, (_, h, d) in zip(vec(p + "conv.b").split(sizes), parts)]))
+        z, x, b, c, dt = mat(p + "in").split([inner] + sizes + [m.heads])
+        return [_pad_rows(z, m.heads, m.vdim)] + [_pad_rows(r, h, d) for r, (_, h, d) in zip((x, b, c), parts)] + [_pad_rows(dt, 1, m.heads)]
+
+    def _pack_attention(self, out: MqhLayer, m: MixerSpec, p: str, mat, vec) -> list:
+        out.kind, out.kv_heads, out.rot, out.scale, out.chunk, out.mix_norm_n = _lib.MQH_ATTENTION, m.kv_heads, m.rot, m.scale, m.chunk, m.dim
+        out.rope = self._rope(m.rot, m.rot_base, m.rot)
+        out.q_bias, out.k_bias = (self._keep(_pad_vec(vec(p + n + ".b"), h, m.dim)) for n, h in (("q", m.heads), ("k", m.kv_heads)))
+        out.q_norm, out.k_norm = (self._keep(_pad_vec(vec(p + n + ".norm"), 1, m.dim)) for n in ("q", "k"))
+        return [_pad_rows(mat(p + "q"), m.heads, m.dim), _pad_rows(mat(p + "k"), m.kv_heads, m.dim), _pad_rows(mat(p + "g"), 1, m.heads)]
+
     def _pack_latent(self, out: MqhLayer, m: MixerSpec, p: str, mat, vec) -> list:
         out.kind, out.mix_norm_n, out.rank, out.rot, out.scale = _lib.MQH_LATENT, m.rank, pad16(m.rank), pad16(m.rot), m.scale
         out.mix_norm = self._keep(_pad_vec(vec(p + "dkv.norm"), 1, m.rank))
         out.sink = self._keep(vec(p + "sink"))
-        key = (m.rot, m.rot_base)
-        if key not in self._ropes:
-            self._ropes[key] = self._keep(interleaved_rope_table(self.max_seq_len_, m.rot, m.rot_base).to(self.device))
-        out.rope = self._ropes[key]
+        out.rope = self._rope(m.rot, m.rot_base, pad16(m.rot))
         uk, uv = _pad_rows(mat(p + "uk"), m.heads, m.dim), _pad_rows(mat(p + "uv"), m.heads, m.vdim)
         w_ukv = torch.cat([_segment(uk), _segment(uv)])
         if w_ukv.shape[0] != self._lib.mqh_ukv_rows(C.byref(out)):

@@ -11,7 +11,7 @@ import os
 from dataclasses import dataclass
 from typing import Callable
 
-from .spec import HybridSpec
+from .spec import DESIGN_MIXERS, HybridSpec
 from .weights import load_hybrid_weights, load_qwen3_weights
 
 
@@ -37,7 +37,7 @@ def _hybrid_decoder(w, max_seq_len, max_prefill_len, dtype, device):
 
 MODELS = {
     "Qwen3ForCausalLM": ModelEntry("Qwen3ForCausalLM", "qwen3", ("bfloat16",), load_qwen3_weights, _qwen3_decoder),
-    "Satosun": ModelEntry("Satosun", "hybrid", ("bfloat16", "float32"), load_hybrid_weights, _hybrid_decoder),
+    **{name: ModelEntry(name, "hybrid", ("bfloat16", "float32"), load_hybrid_weights, _hybrid_decoder) for name in DESIGN_MIXERS},
 }
 
 
@@ -68,7 +68,8 @@ def build_decoder(model_name: str = "Qwen/Qwen3-0.6B", max_seq_len: int = 2048, 
         entry = find_model(model_name)
         weights = entry.load_weights(model_name, max_seq_len=max_seq_len, device=device)
     else:
-        entry = MODELS["Satosun" if isinstance(weights.get("spec"), HybridSpec) else "Qwen3ForCausalLM"]
+        spec = weights.get("spec")
+        entry = MODELS[spec.architecture if isinstance(spec, HybridSpec) else "Qwen3ForCausalLM"]
     if dtype not in entry.dtypes:
         raise ValueError(f"{entry.name} runs in {', '.join(entry.dtypes)}, not {dtype}")
     decoder = entry.make_decoder(weights, max_seq_len, max_seq_len if max_prefill_len is None else max_prefill_len, dtype, device)

@@ -2,9 +2,10 @@
 
 A run is one pass of one layer: a layer that the model loops over has as many
 runs as passes, and each keeps its own.  Two kinds exist: a *cache* with a row
-per position (latents of latent attention), whose rows beyond the position are
-never read and need no clearing, and a *recurrent state* of fixed size
-(lightning attention), which must be zero where a sequence begins.
+per position (latents of latent attention, keys and values), whose rows beyond
+the position are never read and need no clearing, and a *recurrent state* of fixed
+size (lightning attention, gated linear attention, Mamba-2 with the last inputs of
+its convolution), which must be zero where a sequence begins.
 """
 from __future__ import annotations
 

@@ -58,15 +58,25 @@ def random_weights(spec: ModelSpec, max_seq_len: int, seed: int = 0, device="cpu
 
 def random_hybrid_weights(spec: HybridSpec, seed: int = 0, device="cpu") -> dict:
     """Checkpoint tensors of a layer-listed model by name: matrices randn / sqrt(inputs), drawn in the order
-    of ``spec.tensor_shapes()`` from one generator; norms near their neutral value, sinks randn."""
+    of ``spec.tensor_shapes()`` from one generator; norms near their neutral value, sinks randn.  Of mixers whose
+    tokens set the decay: biases such that states live for tens of tokens, step sizes around 0.05."""
     g = torch.Generator().manual_seed(seed)
     tensors = {}
     for name, shape in spec.tensor_shapes().items():
         t = torch.randn(shape, generator=g, dtype=torch.float32)
-        if len(shape) == 2:
+        if name.endswith(("mix.conv", "a2.b", "dt_bias", "A_log", "mix.D")):
+            if name.endswith("mix.conv"):
+                t = t / shape[1] ** 0.5
+            else:
+                low, high = {"a2.b": (0.0, 4.0), "dt_bias": (-5.0, -1.5), "A_log": (0.0, 2.0), "mix.D": (0.5, 1.5)}[
+                    next(k for k in ("a2.b", "dt_bias", "A_log", "mix.D") if name.endswith(k))]
+                t = low + (high - low) * torch.sigmoid(t)
+        elif len(shape) == 2:
             t = t / (shape[1] ** 0.5 if name != "embed" else spec.embed_scale)
-        elif name.endswith(("mix.norm", "dkv.norm")):
+        elif name.endswith(("mix.norm", "dkv.norm", "q.norm", "k.norm")) or (spec.post_norm and "norm" in name):
             t = 1.0 + 0.1 * t
+        elif name.endswith(("ls1", "ls2")):
+            t = 0.7 + 0.2 * t
         elif not name.endswith("sink"):
             t = 0.1 * t                      # stored around zero
         tensors[name] = t.to(torch.bfloat16).to(device)

@@ -61,6 +61,23 @@ def load_tensors(model_dir: str, keys, optional=()) -> dict:
     return out
 
 
+def stored_shapes(model_dir: str) -> dict:
+    """name -> shape of every tensor of the checkpoint, without reading the data."""
+    from safetensors import safe_open
+
+    single = os.path.join(model_dir, "model.safetensors")
+    if os.path.exists(single):
+        files = [single]
+    else:
+        with open(os.path.join(model_dir, "model.safetensors.index.json")) as fh:
+            files = sorted({os.path.join(model_dir, f) for f in json.load(fh)["weight_map"].values()})
+    out = {}
+    for path in files:
+        with safe_open(path, framework="pt", device="cpu") as f:
+            out.update({k: tuple(f.get_slice(k).get_shape()) for k in f.keys()})
+    return out
+
+
 def _bf16(t, device):
     return t.to(torch.bfloat16).contiguous().to(device)
 
@@ -78,7 +95,7 @@ def load_hybrid_weights(model_dir: str, max_seq_len: int = 2048, device="cuda") 
     """Tensors of a layer-listed model by their checkpoint names (on the CPU: the decoder packs them on
     ``device``), with the spec its config.json describes."""
     with open(os.path.join(model_dir, "config.json")) as fh:
-        spec = read_hybrid_config(json.load(fh))
+        spec = read_hybrid_config(json.load(fh), stored_shapes(model_dir))
     shapes = spec.tensor_shapes()
     tensors = load_tensors(model_dir, list(shapes))
     for name, shape in shapes.items():

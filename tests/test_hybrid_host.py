@@ -105,11 +105,11 @@ def test_padding_keeps_products():
 
 
 def test_decay_powers_and_rope_table():
-    from megaqwen_b200.hybrid import decay_powers, interleaved_rope_table
+    from megaqwen_b200.hybrid import decay_powers, rope_table
     d = decay_powers([0.0, 0.5, 0.999, 1.0], 129)
     assert d[:, 0].tolist() == [1.0] * 4 and d[0, 1] == 0 and d[1, 10] == 2.0 ** -10 and d[3, 128] == 1
     assert abs(float(d[2, 128]) - 0.999 ** 128) < 1e-7
-    t = interleaved_rope_table(50, 6, 300.0)
+    t = rope_table(50, 6, 300.0, 16)
     assert t.shape == (50, 8, 2)
     for p, i in ((0, 0), (1, 1), (49, 2)):
         a = p * 300.0 ** (-2 * i / 6)
@@ -137,10 +137,11 @@ def _c_model(max_seq=100):
     one = ctypes.c_void_p(256)            # never dereferenced by the host functions below
     layers = (_lib.MqhLayer * 2)()
     for layer, kind in zip(layers, (_lib.MQH_LATENT, _lib.MQH_LIGHTNING)):
-        layer.kind, layer.heads, layer.dim, layer.vdim, layer.rank, layer.rot, layer.ff, layer.mix_norm_n = kind, 3, 32, 48, 64, 16, 80, 5
+        layer.kind, layer.heads, layer.dim, layer.vdim, layer.rank, layer.rot, layer.ff, layer.mix_norm_n = kind, 3, 32, 48, 64, 16, 80, 126
+        layer.norm_parts, layer.vdim_n = 1, 42
         for n in ("norm", "w_in", "w_out", "mix_norm", "decay_pow", "w_ukv", "w_uk_t", "sink", "rope"):
             setattr(layer, n, one)
-    return _lib.MqhModel(_lib.MQH_BF16, 64, 64, 333, max_seq, 1.0, 1e-6, 1.0, 2, 0, 1, 3, layers, one, one, one, one)
+    return _lib.MqhModel(_lib.MQH_BF16, _lib.MQH_PARALLEL, 64, 64, 333, max_seq, 1.0, 1e-6, 1.0, 2, 0, 1, 3, layers, one, one, one, one)
 
 
 def test_host_entry_points():
@@ -151,8 +152,8 @@ def test_host_entry_points():
     assert lib.mqh_run_count(p) == 4 and [lib.mqh_run_layer(p, r) for r in range(5)] == [0, 0, 0, 1, -1]
     assert lib.mqh_state_bytes(p, 0) == 100 * 80 * 2 and lib.mqh_state_bytes(p, 3) == 3 * 32 * 48 * 4
     assert not lib.mqh_state_recurrent(p, 0) and lib.mqh_state_recurrent(p, 3)
-    assert lib.mqh_in_rows(ctypes.byref(m.layers[0])) == 96 + 64 + 96 + 160
-    assert lib.mqh_in_rows(ctypes.byref(m.layers[1])) == 2 * 96 + 2 * 160 + 160
+    assert lib.mqh_in_rows(ctypes.byref(m.layers[0]), m.form) == 96 + 64 + 96 + 160
+    assert lib.mqh_in_rows(ctypes.byref(m.layers[1]), m.form) == 2 * 96 + 2 * 160 + 160
     assert lib.mqh_ukv_rows(ctypes.byref(m.layers[0])) == 96 + 160 and lib.mqh_ukv_rows(ctypes.byref(m.layers[1])) == 0
     assert lib.mqh_logits_ld(p) == 512
     assert lib.mqh_decode_launch_count(p) == 3 * (1 + 5) + 3 + 1

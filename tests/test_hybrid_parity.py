@@ -356,7 +356,7 @@ def test_lightning_kernels(lib, n, heads, dim, vdim):
     state = torch.randn(heads, dim, vdim, generator=g)
     want, end = lightning_exact(q, k, v, decay, state)
     pw = decay_powers(decay.tolist(), _lib.MQH_CHUNK + 1).cuda()
-    scratch = torch.zeros(lib.mqh_lightning_scratch_bytes(n, heads, dim, vdim), dtype=torch.uint8, device="cuda")
+    scratch = torch.zeros(lib.mqh_recurrence_scratch_bytes(n, heads, dim, vdim), dtype=torch.uint8, device="cuda")
     for code, dt, chunked, tol in ((_lib.MQH_F32, torch.float32, 0, 2e-6), (_lib.MQH_BF16, torch.bfloat16, 0, 2e-6), (_lib.MQH_BF16, torch.bfloat16, 1, 3e-5)):
         a, b, c = (x.to("cuda", dt).contiguous() for x in (q, k, v))
         s, o = state.cuda(), torch.full((n, heads, vdim), float("nan"), device="cuda")
@@ -397,7 +397,7 @@ def test_causal_attention_kernels(lib, n, pos0, heads, dim, rot, vdim):
             out = torch.full((n, heads, vdim), float("nan"), dtype=dt, device="cuda")
             sk = sink.cuda()
             _lib.check(lib.mqh_launch_causal_attention(code, *(x.data_ptr() for x in dev[:4]), ld, dev[4].data_ptr(), sk.data_ptr() if use_sink else None,
-                                                       out.data_ptr(), n, pos0, heads, dim, rot, vdim, scale, tc, status.data_ptr(),
+                                                       None, out.data_ptr(), n, pos0, heads, heads, dim, rot, vdim, 0, scale, tc, status.data_ptr(),
                                                        torch.cuda.current_stream().cuda_stream), "causal")
             err = float((out.double().cpu() - want).abs().max() / want.abs().max())
             assert err < tol and int(status.item()) == 0, (use_sink, dt, tc, err)
@@ -409,7 +409,7 @@ def test_causal_attention_rejects_what_it_does_not_hold(lib):
     p, st = x.data_ptr(), torch.zeros(1, dtype=torch.int32, device="cuda").data_ptr()
 
     def call(dtype, dim, rot, vdim, tc):
-        return lib.mqh_launch_causal_attention(dtype, p, p, p, p, rot, p, None, p, 2, 0, 1, dim, rot, vdim, 1.0, tc, st, None)
+        return lib.mqh_launch_causal_attention(dtype, p, p, p, p, rot, p, None, None, p, 2, 0, 1, 1, dim, rot, vdim, 0, 1.0, tc, st, None)
     assert call(_lib.MQH_BF16, 144, 16, 16, 1) == -3 and call(_lib.MQH_F32, 16, 16, 16, 1) == -3
     assert call(_lib.MQH_BF16, 20, 16, 16, 0) == -1
 
