@@ -75,6 +75,8 @@ def random_hybrid_weights(spec: HybridSpec, seed: int = 0, device="cpu") -> dict
             t = t / (shape[1] ** 0.5 if name != "embed" else spec.embed_scale)
         elif name.endswith(("mix.norm", "dkv.norm", "q.norm", "k.norm")) or (spec.post_norm and "norm" in name):
             t = 1.0 + 0.1 * t
+        elif name.endswith(("q.b", "k.b")):
+            t = 0.5 * t
         elif name.endswith(("ls1", "ls2")):
             t = 0.7 + 0.2 * t
         elif not name.endswith("sink"):
