@@ -446,8 +446,15 @@ def run_ours(args):
 
 def hybrid_spec(name):
     """Layer-listed models at the sizes of real ones (random weights): "0.6b" has the layers, width, heads and
-    vocabulary of Qwen3-0.6B, "0.6b-loop" half of its layers with a stretch that runs twice, "2b" wider layers."""
+    vocabulary of Qwen3-0.6B, "0.6b-loop" half of its layers with a stretch that runs twice, "2b" wider layers; "vunasun-0.6b"
+    and "vunasun-2b" have the same widths and depths with Mamba-2, chunked attention and gated linear attention in turn."""
     from megaqwen_b200.spec import HybridSpec, LayerSpec, MixerSpec
+    if name.startswith("vunasun-"):
+        width, ff, layers = {"0.6b": (1024, 3072, 28), "2b": (2048, 6144, 20)}[name[len("vunasun-"):]]
+        mixers = (MixerSpec("mamba2", 2 * width // 64, 128, 64, kv_heads=1, conv=4, norm_groups=1),
+                  MixerSpec("attention", 16, 128, 128, kv_heads=8, rot=128, rot_base=1e6, scale=128 ** -0.5, chunk=4096),
+                  MixerSpec("gla", 16, 128, 128, tau=16.0, rank=16))
+        return HybridSpec(151936, width, 1.0, 1e-6, 1.0, tuple(LayerSpec(mixers[i % 3], ff) for i in range(layers)), architecture="Vunasun", post_norm=True)
     width, ff, layers, loop = {"0.6b": (1024, 3072, 28, None), "0.6b-loop": (1024, 3072, 14, (2, 12, 2)), "2b": (2048, 6144, 20, None)}[name]
     latent = MixerSpec("latent_attention", 16, 128, 128, rank=512, rot=64, rot_base=1e6, scale=192 ** -0.5)
     light = MixerSpec("lightning", 16, 128, 128, decay=tuple(1.0 - 2.0 ** (-1 - 0.5 * i) for i in range(16)))
@@ -605,7 +612,7 @@ def main():
     ap.add_argument("--ncu-batch", type=int, default=0, help="profiler case: batched decode steps with this batch size")
     ap.add_argument("--ncu-persistent", action="store_true", help="profiler case runs the persistent chain kernel")
     ap.add_argument("--hybrid", action="store_true", help="measure layer-listed models beside Qwen3-0.6B instead of the headline workload")
-    ap.add_argument("--hybrid-sizes", default="qwen3-0.6b,0.6b,0.6b-loop,2b", help="models of --hybrid, with commas between them")
+    ap.add_argument("--hybrid-sizes", default="qwen3-0.6b,0.6b,0.6b-loop,2b,vunasun-0.6b,vunasun-2b", help="models of --hybrid, with commas between them")
     args = ap.parse_args()
     if args.hybrid:
         run_hybrid(args)

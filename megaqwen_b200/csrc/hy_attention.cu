@@ -75,7 +75,7 @@ template int attn_rows<bf16>(Stream&, const AttnRowsArgs&);
 template int attn_rows<float>(Stream&, const AttnRowsArgs&);
 
 // ---------------------------------------------------------------- one token: what both kernels share
-constexpr int AD_KEYS = 64;
+constexpr int AD_KEYS = 16;
 struct Piece { int pos, first, kbeg, kend; };            // keys [kbeg, kend) of the visible [first, pos]
 // the position was set before this step began
 __device__ __forceinline__ Piece my_piece(const AttnDecodeArgs& a) {
@@ -124,35 +124,39 @@ __device__ __forceinline__ void merge_pieces(const AttnDecodeArgs& a, const floa
 }
 
 // ---------------------------------------------------------------- one token: bf16
-// Grid (pieces, key heads, groups of sixteen query heads), a cluster per (y, z).
-constexpr int AD_THREADS = 256, AD_WARPS = 8, AD_MAXT = 4, AD_PLD = AD_KEYS + 8;
-constexpr int AD_MAX_DIM = AD_MAXT * 64;
+// Grid (pieces, key heads, groups of sixteen query heads), a cluster per (y, z).  Every warp takes sixteen keys at a time
+// through its own stages of shared memory and keeps its own maximum, sum and output, so that no tile needs a barrier; the
+// weights of a tile stay in registers as the A operand of the second product.  The warps meet once, at the end.
+// NT: 8-column tiles of the output, dim <= 8 NT.
+constexpr int AD_THREADS = 256, AD_WARPS = 8;
+constexpr int AD_MAX_DIM = 256;
 static size_t ad_smem(int dim, int stages) {
-    return (size_t)(stages * 2 * AD_KEYS + 16 + 2) * (dim + 8) * 2 + (size_t)AD_WARPS * dim * 4 + (size_t)16 * dim * 4;
+    return (size_t)(AD_WARPS * stages * 2 * AD_KEYS + 16 + 2) * (dim + 8) * 2 + (size_t)AD_WARPS * dim * 4 + (size_t)16 * dim * 4;
 }
-template <int STAGES>
+template <int NT, int STAGES>
 __global__ void __launch_bounds__(AD_THREADS) k_attn_decode(AttnDecodeArgs a) {
     extern __shared__ __align__(16) uint8_t ad_raw[];
-    __shared__ __align__(16) bf16 sp[16 * AD_PLD];
-    __shared__ float smax[AD_WARPS][16], ssum[AD_WARPS][16], ml[32];
+    __shared__ float wm[AD_WARPS][16], wl[AD_WARPS][16], ml[32];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, dim = a.qn.dim, ld = dim + 8, d8 = dim / 8;
-    bf16* sk = reinterpret_cast<bf16*>(ad_raw);          // [STAGES][keys, then values][AD_KEYS][ld]
-    bf16* sq = sk + STAGES * 2 * AD_KEYS * ld;           // [16][ld]
+    bf16* stages = reinterpret_cast<bf16*>(ad_raw);      // [warps][STAGES][keys, then values][AD_KEYS][ld]
+    bf16* mine = stages + warp * STAGES * 2 * AD_KEYS * ld;
+    bf16* sq = stages + AD_WARPS * STAGES * 2 * AD_KEYS * ld;    // [16][ld]
     bf16* snew = sq + 16 * ld;                           // key and value of the token itself
     float* buf = reinterpret_cast<float*>(snew + 2 * ld);    // [warps][dim]
     float* sacc = buf + AD_WARPS * dim;                  // [16][dim]
     const int g = blockIdx.y, group = a.heads / a.kv_heads, h0 = g * group + blockIdx.z * 16, nh = min(16, group - (int)blockIdx.z * 16);
     const Piece pc = my_piece(a);
-    const int ntiles = pc.kend > pc.kbeg ? (pc.kend - pc.kbeg + AD_KEYS - 1) / AD_KEYS : 0;
-    const bool has_new = ntiles > 0 && pc.kend == pc.pos + 1;
+    const int tiles = pc.kend > pc.kbeg ? (pc.kend - pc.kbeg + AD_KEYS - 1) / AD_KEYS : 0;
+    const int count = tiles > warp ? (tiles - warp + AD_WARPS - 1) / AD_WARPS : 0;       // this warp's tiles: warp, warp + 8, ..
+    const bool has_new = tiles > 0 && pc.kend == pc.pos + 1;
     const bf16 *kc = reinterpret_cast<const bf16*>(a.k_cache) + (size_t)g * dim, *vc = reinterpret_cast<const bf16*>(a.v_cache) + (size_t)g * dim;
     const size_t row = (size_t)a.kv_heads * dim;
     // A tile's cached rows; those beyond the piece become zeros, that of the token itself is left out
-    auto fetch = [&](int t) {
-        if (t < ntiles) {
-            bf16* dst = sk + (t % STAGES) * 2 * AD_KEYS * ld;
-            const int k0 = pc.kbeg + t * AD_KEYS;
-            for (int x = tid; x < AD_KEYS * d8; x += AD_THREADS) {
+    auto fetch = [&](int i) {
+        if (i < count) {
+            bf16* dst = mine + (i % STAGES) * 2 * AD_KEYS * ld;
+            const int k0 = pc.kbeg + (warp + i * AD_WARPS) * AD_KEYS;
+            for (int x = lane; x < AD_KEYS * d8; x += 32) {
                 const int j = x / d8, col = (x - j * d8) * 8, key = k0 + j;
                 if (key == pc.pos) continue;
                 const bool ok = key < pc.kend;
@@ -164,20 +168,18 @@ __global__ void __launch_bounds__(AD_THREADS) k_attn_decode(AttnDecodeArgs a) {
     };
     pdl_trigger();
 #pragma unroll
-    for (int t = 0; t < STAGES; ++t) fetch(t);
+    for (int i = 0; i < STAGES; ++i) fetch(i);
     pdl_wait_cta();
     const float2* rope = reinterpret_cast<const float2*>(a.qn.rope) + (size_t)pc.pos * a.qn.half;
     const bf16* knew = reinterpret_cast<const bf16*>(a.k) + (size_t)g * dim;
-    for (int x = warp; x < 16 + (has_new ? 1 : 0); x += AD_WARPS) {
+    // query rows 0 .. nh - 1, the new key as row nh; the remaining rows of the product are zeros
+    for (int x = warp; x < nh + (has_new ? 1 : 0); x += AD_WARPS) {
         float* b = buf + warp * dim;
-        bf16* dst = x < 16 ? sq + x * ld : snew;
-        if (x >= nh && x < 16) {
-            for (int i = lane * 4; i < dim; i += 128) store4(dst + i, make_float4(0.f, 0.f, 0.f, 0.f));
-            continue;
-        }
-        norm_rotate(x < 16 ? reinterpret_cast<const bf16*>(a.q) + (size_t)(h0 + x) * dim : knew, x < 16 ? a.qn : a.kn, rope, b);
+        const bool key = x == nh;
+        bf16* dst = key ? snew : sq + x * ld;
+        norm_rotate(key ? knew : reinterpret_cast<const bf16*>(a.q) + (size_t)(h0 + x) * dim, key ? a.kn : a.qn, rope, b);
         for (int i = lane * 4; i < dim; i += 128) store4(dst + i, load4(b + i));
-        if (x == 16)
+        if (key)
             for (int i = lane * 4; i < dim; i += 128) {
                 const float4 v = load4_cg(knew + i);
                 store4(snew + ld + i, v);
@@ -188,118 +190,128 @@ __global__ void __launch_bounds__(AD_THREADS) k_attn_decode(AttnDecodeArgs a) {
             }
         __syncwarp();
     }
+    for (int x = tid; x < (16 - nh) * d8; x += AD_THREADS)
+        *reinterpret_cast<uint4*>(sq + (nh + x / d8) * ld + (x % d8) * 8) = make_uint4(0u, 0u, 0u, 0u);
     __syncthreads();
     const float c = a.scale * LOG2E;
-    const int nt8 = dim / 8, tpw = 2 * ((nt8 + 15) / 16), tile0 = warp * tpw;      // this warp's 8-column tiles of the output
-    float acc[AD_MAXT][4];
+    float acc[NT][4];
 #pragma unroll
-    for (int i = 0; i < AD_MAXT; ++i)
+    for (int i = 0; i < NT; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};               // rows lane / 4, lane / 4 + 8
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};               // rows lane / 4, lane / 4 + 8; l: this lane's keys
     const int r = lane >> 2;
     const uint32_t qa = smem_u32(sq + (lane & 15) * ld + (lane >> 4) * 8);
-    for (int t = 0; t < ntiles; ++t) {
-        bf16 *tk = sk + (t % STAGES) * 2 * AD_KEYS * ld, *tv = tk + AD_KEYS * ld;
-        const int k0 = pc.kbeg + t * AD_KEYS;
+    const int koff = ((lane & 7) + ((lane >> 4) & 1) * 8) * ld + ((lane >> 3) & 1) * 8, voff = (AD_KEYS + (lane & 15)) * ld + (lane >> 4) * 8;
+    for (int i = 0; i < count; ++i) {
+        bf16* tile = mine + (i % STAGES) * 2 * AD_KEYS * ld;
+        const int k0 = pc.kbeg + (warp + i * AD_WARPS) * AD_KEYS;
         cp_async_wait<STAGES - 1>();
-        if (has_new && t == ntiles - 1 && tid < 2 * d8) {
-            const int j = pc.pos - k0, col = (tid % d8) * 8;
-            *reinterpret_cast<uint4*>((tid < d8 ? tk : tv) + j * ld + col) = *reinterpret_cast<const uint4*>((tid < d8 ? snew : snew + ld) + col);
-        }
-        __syncthreads();
-        // scores of this warp's eight keys
-        float s0[4] = {}, s1[4] = {};
-        const uint32_t kb = smem_u32(tk + (warp * 8 + r) * ld + (lane & 3) * 2);
+        if (pc.pos >= k0 && pc.pos < k0 + AD_KEYS)       // the token itself (in the last piece only)
+            for (int x = lane; x < 2 * d8; x += 32) {
+                const bool val = x >= d8;
+                *reinterpret_cast<uint4*>(tile + ((val ? AD_KEYS : 0) + pc.pos - k0) * ld + (x % d8) * 8) =
+                    *reinterpret_cast<const uint4*>(snew + (val ? ld : 0) + (x % d8) * 8);
+            }
+        __syncwarp();
+        float s0[2][4] = {}, s1[2][4] = {};              // scores of keys 0-7, 8-15; two sums each break the chain of products
+        const uint32_t ka = smem_u32(tile + koff);
         int ks = 0;
 #pragma unroll 4
         for (; ks + 1 < dim / 16; ks += 2) {
-            uint32_t q4[4], r4[4];
-            ldsm4(q4, qa + ks * 32);
-            ldsm4(r4, qa + ks * 32 + 32);
-            mma16816(s0, q4, lds32(kb + ks * 32), lds32(kb + ks * 32 + 16));
-            mma16816(s1, r4, lds32(kb + ks * 32 + 32), lds32(kb + ks * 32 + 48));
+            uint32_t q0[4], q1[4], b0[4], b1[4];
+            ldsm4(q0, qa + ks * 32);
+            ldsm4(b0, ka + ks * 32);
+            ldsm4(q1, qa + ks * 32 + 32);
+            ldsm4(b1, ka + ks * 32 + 32);
+            mma16816(s0[0], q0, b0[0], b0[1]);
+            mma16816(s0[1], q0, b0[2], b0[3]);
+            mma16816(s1[0], q1, b1[0], b1[1]);
+            mma16816(s1[1], q1, b1[2], b1[3]);
         }
         if (ks < dim / 16) {
-            uint32_t q4[4];
-            ldsm4(q4, qa + ks * 32);
-            mma16816(s0, q4, lds32(kb + ks * 32), lds32(kb + ks * 32 + 16));
+            uint32_t q0[4], b0[4];
+            ldsm4(q0, qa + ks * 32);
+            ldsm4(b0, ka + ks * 32);
+            mma16816(s0[0], q0, b0[0], b0[1]);
+            mma16816(s0[1], q0, b0[2], b0[3]);
         }
-        float s[4];
+        float s[2][4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int key = k0 + warp * 8 + 2 * (lane & 3) + (e & 1);
-            s[e] = key < pc.kend ? (s0[e] + s1[e]) * c : -INFINITY;
-        }
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[n][e] = k0 + n * 8 + 2 * (lane & 3) + (e & 1) < pc.kend ? (s0[n][e] + s1[n][e]) * c : -INFINITY;
+        uint32_t p4[4];
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
-            float v = fmaxf(s[2 * h], s[2 * h + 1]);
+            float v = fmaxf(fmaxf(s[0][2 * h], s[0][2 * h + 1]), fmaxf(s[1][2 * h], s[1][2 * h + 1]));
             v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 1));
             v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 2));
-            if ((lane & 3) == 0) smax[warp][r + 8 * h] = v;
-        }
-        __syncthreads();
-        float alpha[2];
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-            float mn = m[h];
-#pragma unroll
-            for (int w = 0; w < AD_WARPS; ++w) mn = fmaxf(mn, smax[w][r + 8 * h]);      // finite: every tile has a key
-            alpha[h] = exp2f(m[h] - mn);
+            const float mn = fmaxf(m[h], v), alpha = exp2f(m[h] - mn);   // finite: every tile has a key
             m[h] = mn;
-            const float p0 = exp2f(s[2 * h] - mn), p1 = exp2f(s[2 * h + 1] - mn);
-            *reinterpret_cast<uint32_t*>(sp + (r + 8 * h) * AD_PLD + warp * 8 + 2 * (lane & 3)) = pack_bf16x2(p0, p1);
-            float v = p0 + p1;
-            v += __shfl_xor_sync(0xffffffffu, v, 1);
-            v += __shfl_xor_sync(0xffffffffu, v, 2);
-            if ((lane & 3) == 0) ssum[warp][r + 8 * h] = v;
+            const float p0 = exp2f(s[0][2 * h] - mn), p1 = exp2f(s[0][2 * h + 1] - mn), p2 = exp2f(s[1][2 * h] - mn), p3 = exp2f(s[1][2 * h + 1] - mn);
+            l[h] = l[h] * alpha + (p0 + p1) + (p2 + p3);
+            p4[h] = pack_bf16x2(p0, p1);
+            p4[2 + h] = pack_bf16x2(p2, p3);
+#pragma unroll
+            for (int n = 0; n < NT; ++n) { acc[n][2 * h] *= alpha; acc[n][2 * h + 1] *= alpha; }
         }
-        __syncthreads();
+        const uint32_t va = smem_u32(tile + voff);
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
-            float v = 0.f;
-#pragma unroll
-            for (int w = 0; w < AD_WARPS; ++w) v += ssum[w][r + 8 * h];
-            l[h] = l[h] * alpha[h] + v;
+        for (int n = 0; n < NT; n += 2) {
+            if (n * 8 >= dim) break;
+            uint32_t b[4];
+            ldsm4_t(b, va + n * 16);
+            mma16816(acc[n], p4, b[0], b[1]);
+            mma16816(acc[n + 1], p4, b[2], b[3]);
         }
-#pragma unroll
-        for (int i = 0; i < AD_MAXT; ++i) { acc[i][0] *= alpha[0]; acc[i][1] *= alpha[0]; acc[i][2] *= alpha[1]; acc[i][3] *= alpha[1]; }
-#pragma unroll
-        for (int ks2 = 0; ks2 < AD_KEYS / 16; ++ks2) {
-            uint32_t p4[4];
-            ldsm4(p4, smem_u32(sp + (lane & 15) * AD_PLD + ks2 * 16 + (lane >> 4) * 8));
-#pragma unroll
-            for (int i = 0; i < AD_MAXT; i += 2) {
-                if (i >= tpw || tile0 + i >= nt8) break;
-                uint32_t b[4];
-                ldsm4_t(b, smem_u32(tv + (ks2 * 16 + (lane & 15)) * ld + (tile0 + i) * 8 + (lane >> 4) * 8));
-                mma16816(acc[i], p4, b[0], b[1]);
-                mma16816(acc[i + 1], p4, b[2], b[3]);
-            }
-        }
-        __syncthreads();                                   // the stage, the weights and the maxima are overwritten next
-        fetch(t + STAGES);
+        __syncwarp();                                      // the stage is overwritten next
+        fetch(i + STAGES);
     }
     cp_async_wait_all();
+    __syncwarp();
+    float* wacc = reinterpret_cast<float*>(mine);          // [16][dim] over this warp's stages
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
+        l[h] += __shfl_xor_sync(0xffffffffu, l[h], 1);
+        l[h] += __shfl_xor_sync(0xffffffffu, l[h], 2);
+        const int x = r + 8 * h;
+        if ((lane & 3) == 0) { wm[warp][x] = m[h]; wl[warp][x] = l[h]; }
+        if (x < nh) {
 #pragma unroll
-        for (int i = 0; i < AD_MAXT; ++i) {
-            if (i >= tpw || tile0 + i >= nt8) break;
-            *reinterpret_cast<float2*>(sacc + (r + 8 * h) * dim + (tile0 + i) * 8 + 2 * (lane & 3)) = make_float2(acc[i][2 * h], acc[i][2 * h + 1]);
+            for (int n = 0; n < NT; ++n) {
+                if (n * 8 >= dim) break;
+                *reinterpret_cast<float2*>(wacc + x * dim + n * 8 + 2 * (lane & 3)) = make_float2(acc[n][2 * h], acc[n][2 * h + 1]);
+            }
         }
-        if (warp == 0 && (lane & 3) == 0) { ml[2 * (r + 8 * h)] = m[h]; ml[2 * (r + 8 * h) + 1] = l[h]; }
+    }
+    __syncthreads();
+    // the warps' shares -> this CTA's; one without keys has the maximum -inf and weighs nothing
+    for (int x = tid; x < nh * dim; x += AD_THREADS) {
+        const int y = x / dim;
+        float mx = -INFINITY, lsum = 0.f, sum = 0.f;
+#pragma unroll
+        for (int w = 0; w < AD_WARPS; ++w) mx = fmaxf(mx, wm[w][y]);
+        if (mx > -INFINITY)
+#pragma unroll
+            for (int w = 0; w < AD_WARPS; ++w) {
+                const float f = exp2f(wm[w][y] - mx);
+                lsum = fmaf(f, wl[w][y], lsum);
+                sum = fmaf(f, reinterpret_cast<const float*>(stages + w * STAGES * 2 * AD_KEYS * ld)[x], sum);
+            }
+        sacc[x] = sum;
+        if (x == y * dim) { ml[2 * y] = mx; ml[2 * y + 1] = lsum; }
     }
     merge_pieces<bf16, AD_THREADS>(a, sacc, ml, nh, h0, dim);
 }
 
 // ---------------------------------------------------------------- one token: 32-bit caches, larger heads
 // Grid (pieces, query heads), a cluster per head; a warp per key, then a thread per column.
-constexpr int AP_THREADS = 128, AP_MAXC = 4;
+constexpr int AP_THREADS = 128, AP_MAXC = 4, AP_KEYS = 64;
 template <typename T>
 __global__ void __launch_bounds__(AP_THREADS) k_attn_decode_plain(AttnDecodeArgs a) {
     extern __shared__ float ap_buf[];                      // query, key of the token itself, output: [dim] each
-    __shared__ float p[AD_KEYS], red[4], ml[2];
+    __shared__ float p[AP_KEYS], red[4], ml[2];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, dim = a.qn.dim, head = blockIdx.y, group = a.heads / a.kv_heads, g = head / group;
     float *sq = ap_buf, *snew = ap_buf + dim, *sacc = ap_buf + 2 * dim;
     pdl_trigger();
@@ -326,8 +338,8 @@ __global__ void __launch_bounds__(AP_THREADS) k_attn_decode_plain(AttnDecodeArgs
     __syncthreads();
     const float c = a.scale * LOG2E;
     float m = -INFINITY, l = 0.f, acc[AP_MAXC] = {};
-    for (int k0 = pc.kbeg; k0 < pc.kend; k0 += AD_KEYS) {
-        const int cnt = min(AD_KEYS, pc.kend - k0);
+    for (int k0 = pc.kbeg; k0 < pc.kend; k0 += AP_KEYS) {
+        const int cnt = min(AP_KEYS, pc.kend - k0);
         float best = -INFINITY;
         for (int j = warp; j < cnt; j += 4) {
             const bool self = k0 + j == pc.pos;
@@ -372,16 +384,17 @@ __global__ void __launch_bounds__(AP_THREADS) k_attn_decode_plain(AttnDecodeArgs
 template <typename T>
 int attn_decode(Stream& st, const AttnDecodeArgs& a) {
     const int dim = a.qn.dim, most = a.chunk > 0 && a.chunk < a.max_seq ? a.chunk : a.max_seq;
-    const int tiles = (most + AD_KEYS - 1) / AD_KEYS, pieces = tiles >= 8 ? 8 : tiles >= 4 ? 4 : tiles >= 2 ? 2 : 1;
+    // one piece per 64 keys that a position may see, up to the portable cluster size
+    const int tiles = (most + 63) / 64, pieces = tiles >= 8 ? 8 : tiles >= 4 ? 4 : tiles >= 2 ? 2 : 1;
     if (sizeof(T) == 2 && dim <= AD_MAX_DIM) {
         const dim3 grid(pieces, a.kv_heads, (a.heads / a.kv_heads + 15) / 16);
-        const int per = (tiles + pieces - 1) / pieces;
-        if (per >= 3 && ad_smem(dim, 4) <= 200 * 1024) {
-            const int rc = allow_smem(k_attn_decode<4>, ad_smem(dim, 4));
-            return rc ? rc : launch_cluster(st, k_attn_decode<4>, grid, dim3(AD_THREADS), ad_smem(dim, 4), pieces, a);
-        }
-        const int rc = allow_smem(k_attn_decode<2>, ad_smem(dim, 2));
-        return rc ? rc : launch_cluster(st, k_attn_decode<2>, grid, dim3(AD_THREADS), ad_smem(dim, 2), pieces, a);
+        auto go = [&](auto kernel, int stages) {
+            const int rc = allow_smem(kernel, ad_smem(dim, stages));
+            return rc ? rc : launch_cluster(st, kernel, grid, dim3(AD_THREADS), ad_smem(dim, stages), pieces, a);
+        };
+        if (dim <= 64) return go(k_attn_decode<8, 3>, 3);
+        if (dim <= 128) return go(k_attn_decode<16, 2>, 2);
+        return go(k_attn_decode<32, 1>, 1);
     }
     if (dim > AP_MAXC * AP_THREADS) return MQ_ERR_UNSUPPORTED;
     return launch_cluster(st, k_attn_decode_plain<T>, dim3(pieces, a.heads), dim3(AP_THREADS), (size_t)dim * 12, pieces, a);

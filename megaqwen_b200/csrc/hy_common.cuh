@@ -129,8 +129,15 @@ struct GatedNorm {
 };
 // squares are kept per unit of four elements where no part ends inside one, else per element
 __host__ __device__ __forceinline__ int gated_unit(const GatedNorm& a) { return (a.vd | a.part_n) % 4 == 0 ? 4 : 1; }
-// floats of shared memory beside the hv of the values; none for one part
-__host__ __device__ __forceinline__ int gated_scratch(const GatedNorm& a) { return a.parts == 1 ? 0 : a.hv / gated_unit(a) + a.parts + 64; }
+// quads of a part where parts are neighbouring lanes of a warp (no padding, a power of two up to 32 quads), else 0
+__host__ __device__ __forceinline__ int gated_lanes(const GatedNorm& a) {
+    const int n = a.part_n / 4;
+    return a.vd == a.vp && a.part_n % 4 == 0 && n <= 32 && (n & (n - 1)) == 0 ? n : 0;
+}
+// floats of shared memory beside the hv of the values; none for one part, or parts inside a warp
+__host__ __device__ __forceinline__ int gated_scratch(const GatedNorm& a) {
+    return a.parts == 1 || gated_lanes(a) ? 0 : a.hv / gated_unit(a) + a.parts + 64;
+}
 template <typename T>
 __device__ __forceinline__ float gate_act(int act, float z) { return act == GATE_SILU ? silu<T>(z) : Elem<T>::sigmoid(z); }
 // One row by a CTA of NW warps.  raw: hv floats, scratch: gated_scratch floats, red: NW floats (all shared); out: T [hv] (may be
@@ -140,33 +147,45 @@ __device__ __forceinline__ void gated_norm_row(const GatedNorm& a, const float4 
     constexpr int STRIDE = NW * 128;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const T* gate = reinterpret_cast<const T*>(a.g);
-    const int unit = gated_unit(a);
+    const int unit = gated_unit(a), lanes = gated_lanes(a);
     float ss = 0.f;
     int n = 0;
-    for (int i0 = tid * 4; i0 < a.hv; i0 += 2 * STRIDE, n += 2) {
+    // whole warps go round: lanes beyond the end take part in the exchanges with zeros
+    for (int i0 = tid * 4; (i0 & ~127) < a.hv; i0 += 2 * STRIDE, n += 2) {
         float4 v[2], g[2];
 #pragma unroll
         for (int x = 0; x < 2; ++x) {
             const int i = i0 + x * STRIDE;
-            if (i >= a.hv) break;
+            v[x] = g[x] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i >= a.hv) continue;
             v[x] = load4_cg(a.o + i);
             g[x] = load4_cg(gate + i);
         }
 #pragma unroll
         for (int x = 0; x < 2; ++x) {
             const int i = i0 + x * STRIDE;
-            if (i >= a.hv) break;
-            const float4 w = n == 0 ? w0[x] : load4(a.w + i);
+            if ((i & ~127) >= a.hv) break;
+            const bool in = i < a.hv;
+            const float4 w = !in ? make_float4(0.f, 0.f, 0.f, 0.f) : n == 0 ? w0[x] : load4(a.w + i);
             const float4 s = make_float4(gate_act<T>(a.act, g[x].x), gate_act<T>(a.act, g[x].y), gate_act<T>(a.act, g[x].z), gate_act<T>(a.act, g[x].w));
             const float4 u = make_float4(v[x].x * s.x, v[x].y * s.y, v[x].z * s.z, v[x].w * s.w);
             const float4 m = a.gate_first ? u : v[x];
             const float4 q = make_float4(m.x * m.x, m.y * m.y, m.z * m.z, m.w * m.w);
+            if (lanes) {
+                float t = q.x + q.y + q.z + q.w;
+                for (int o = lanes >> 1; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+                const float inv = 1.0f / sqrtf(t / (float)a.part_n + a.eps);
+                if (in) store4(out + i, make_float4(u.x * w.x * inv, u.y * w.y * inv, u.z * w.z * inv, u.w * w.w * inv));
+                continue;
+            }
+            if (!in) continue;
             if (a.parts == 1) ss += q.x + q.y + q.z + q.w;
             else if (unit == 4) scratch[i >> 2] = q.x + q.y + q.z + q.w;
             else store4(scratch + i, q);
             store4(raw + i, make_float4(u.x * w.x, u.y * w.y, u.z * w.z, u.w * w.w));
         }
     }
+    if (lanes) return;
     if (a.parts == 1) {
         const float inv = 1.0f / sqrtf(cta_sum<NW>(ss, red) / (float)a.part_n + a.eps);
         for (int i = tid * 4; i < a.hv; i += STRIDE) {

@@ -40,24 +40,29 @@ __device__ __forceinline__ void mma_row(float (&acc)[2 * NP][4], const uint32_t 
 
 // log2 of the factor sigmoid(z)^inv_tau
 __device__ __forceinline__ float channel_log_decay(float z, float inv_tau) { return -softplus(-z) * inv_tau * LOG2E; }
+// the same by base-2 functions; 1 + e is rounded, an error of 2^-24 in the factor before it is raised to inv_tau
+__device__ __forceinline__ float channel_log_decay_fast(float z, float inv_tau) {
+    return -fmaf(fmaxf(-z, 0.f), LOG2E, log2f(1.0f + exp2f(-fabsf(z) * LOG2E))) * inv_tau;
+}
 
 // ---------------------------------------------------------------- short convolution
 // y_t = silu(b + sum_j w[j] x_(t - taps + 1 + j)), channel by channel.  The state holds the input of position p in row p % taps:
 // a token reads the taps - 1 rows before its own and overwrites the one row that nobody needs any more.  Positions before 0
 // count as zeros, so a new sequence needs no clearing.
 __device__ __forceinline__ int ring_row(int pos, int taps) { return pos % taps; }
-constexpr int CV_THREADS = 256, CV_TOKENS = CONV_MAX_TAPS;     // tokens of one CTA: only the first CTA looks before the portion
+constexpr int CV_THREADS = 512, CV_RUN = 8, CV_TOKENS = CONV_MAX_TAPS;     // tokens of one CTA: only the first CTA looks before the portion
+static_assert(CV_THREADS / 64 * CV_RUN == CV_TOKENS, "runs of a CTA");
 template <typename T>
 __global__ void __launch_bounds__(CV_THREADS) k_conv_rows(const T* __restrict__ x, const float* __restrict__ w, const float* __restrict__ b, T* state,
                                                           T* __restrict__ y, int n, int pos0, int channels, int taps) {
     pdl_trigger();
     pdl_wait();
-    const int c = (blockIdx.x * (CV_THREADS / 4) + (threadIdx.x & 63)) * 4, t0 = blockIdx.y * CV_TOKENS, t1 = min(t0 + CV_TOKENS, n);
+    const int c = (blockIdx.x * 64 + (threadIdx.x & 63)) * 4, t0 = blockIdx.y * CV_TOKENS, t1 = min(t0 + CV_TOKENS, n);
     const bool live = c < channels;
     if (live) {
         const float4 bias = load4(b + c);
-        // four runs of tokens per CTA; a run's inputs move through a window of at most four registers, longer filters read again
-        const int per = CV_TOKENS / 4, ta = t0 + (threadIdx.x >> 6) * per, te = min(ta + per, t1);
+        // a thread has a run of eight tokens; with four taps its inputs are read once, side by side, other filters read again
+        const int ta = t0 + (threadIdx.x >> 6) * CV_RUN, te = min(ta + CV_RUN, t1);
         auto input = [&](int t) {
             if (t >= 0) return load4_cg(x + (size_t)t * channels + c);
             if (pos0 + t < 0) return make_float4(0.f, 0.f, 0.f, 0.f);
@@ -71,15 +76,17 @@ __global__ void __launch_bounds__(CV_THREADS) k_conv_rows(const T* __restrict__ 
         };
         if (taps == 4 && ta < te) {
             const float4 w0 = load4(w + c), w1 = load4(w + channels + c), w2 = load4(w + 2 * channels + c), w3 = load4(w + 3 * channels + c);
-            float4 a0 = input(ta - 3), a1 = input(ta - 2), a2 = input(ta - 1);
-#pragma unroll 4
-            for (int t = ta; t < te; ++t) {
-                const float4 a3 = input(t);
-                float4 s = bias;
-                add(s, w0, a0); add(s, w1, a1); add(s, w2, a2); add(s, w3, a3);
-                put(t, s);
-                a0 = a1; a1 = a2; a2 = a3;
-            }
+            float4 in[CV_RUN + 3];
+#pragma unroll
+            for (int i = 0; i < CV_RUN + 3; ++i)
+                if (ta + i - 3 < te) in[i] = input(ta + i - 3);
+#pragma unroll
+            for (int i = 0; i < CV_RUN; ++i)
+                if (ta + i < te) {
+                    float4 s = bias;
+                    add(s, w0, in[i]); add(s, w1, in[i + 1]); add(s, w2, in[i + 2]); add(s, w3, in[i + 3]);
+                    put(ta + i, s);
+                }
         } else {
             for (int t = ta; t < te; ++t) {
                 float4 s = bias;
@@ -299,14 +306,15 @@ __device__ __forceinline__ void copy_tile(bf16* dst, int sld, const bf16* src, s
 }
 
 // ---------------------------------------------------------------- chunked: decays
-// Per head: step sizes dt and running sums (inclusive) of the log2 decays of a chunk's tokens; tokens beyond cnt add nothing.
-// Every thread of the CTA calls it; the results stand behind a barrier.
+// Per head: step sizes dt and running sums (inclusive) of the log2 decays of a chunk's tokens, [HP][LC] for heads head ..;
+// tokens beyond cnt add nothing.  Every thread of the CTA calls it; the results stand behind a barrier.
+template <int HP>
 __device__ __forceinline__ void head_decays(const RecurrenceArgs& a, int head, size_t row0, int cnt, float* dt, float* L, float* wsum) {
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, t = tid & (LC - 1), h = head + tid / LC;
     float x = 0.f, s = 0.f;
-    if (tid < LC) {
-        if (tid < cnt) x = softplus(__ldcg(a.decay_in + (row0 + tid) * a.ld_decay + head) + a.dt_bias[head]);
-        s = x * a.a_neg[head] * LOG2E;
+    if (tid < HP * LC) {
+        if (t < cnt) x = softplus(__ldcg(a.decay_in + (row0 + t) * a.ld_decay + h) + a.dt_bias[h]);
+        s = x * a.a_neg[h] * LOG2E;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const float u = __shfl_up_sync(0xffffffffu, s, o);
@@ -315,17 +323,27 @@ __device__ __forceinline__ void head_decays(const RecurrenceArgs& a, int head, s
         if (lane == 31) wsum[warp] = s;
     }
     __syncthreads();
-    if (tid < LC) {
-        for (int w = 0; w < warp; ++w) s += wsum[w];
+    if (tid < HP * LC) {
+        for (int w = warp & ~(LC / 32 - 1); w < warp; ++w) s += wsum[w];
         dt[tid] = x;
         L[tid] = s;
     }
     __syncthreads();
 }
+// value columns (v or the state): JT columns of one head, or 64 each of two heads whose columns are `next` elements apart
+template <int THREADS, int JT, bool PAIR>
+__device__ __forceinline__ void copy_values(bf16* dst, const bf16* src, size_t ld, int rows, int live, int cols_live, size_t next) {
+    if (PAIR) {
+        copy_tile<THREADS, 8>(dst, JT + 8, src, ld, rows, live, 64, cols_live);
+        copy_tile<THREADS, 8>(dst + 64, JT + 8, src + next, ld, rows, live, 64, cols_live);
+    } else {
+        copy_tile<THREADS, JT / 8>(dst, JT + 8, src, ld, rows, live, JT, cols_live);
+    }
+}
 // Per key channel: cum [n, heads*dim] = running sums (inclusive, from the chunk's first token) of the log2 decays.
 // One CTA per (32 channels, chunk): thread = (channel, run of CG_RUN tokens).
-constexpr int CG_RUN = 8, CG_THREADS = 32 * (LC / CG_RUN), CG_RANK = 16;
-__global__ void __launch_bounds__(CG_THREADS) k_channel_decays(RecurrenceArgs a, float* __restrict__ cum) {
+constexpr int CG_RUN = 16, CG_THREADS = 32 * (LC / CG_RUN), CG_RANK = 16;
+__global__ void __launch_bounds__(CG_THREADS, 4) k_channel_decays(RecurrenceArgs a, float* __restrict__ cum) {
     pdl_trigger();
     __shared__ float in[LC][CG_RANK];
     __shared__ float total[LC / CG_RUN][32];
@@ -338,12 +356,16 @@ __global__ void __launch_bounds__(CG_THREADS) k_channel_decays(RecurrenceArgs a,
     float z[CG_RUN];
 #pragma unroll
     for (int x = 0; x < CG_RUN; ++x) z[x] = b;
+    float w[CG_RANK];
+#pragma unroll
+    for (int r = 0; r < CG_RANK; ++r) w[r] = live ? __bfloat162float(gw[(size_t)r * a.dim]) : 0.f;
     pdl_wait();
     for (int r0 = 0; r0 < a.rank; r0 += CG_RANK) {         // rank is a multiple of 16
-        float w[CG_RANK];
+        if (r0 > 0) {
 #pragma unroll
-        for (int r = 0; r < CG_RANK; ++r) w[r] = live ? __bfloat162float(gw[(size_t)(r0 + r) * a.dim]) : 0.f;
-        __syncthreads();
+            for (int r = 0; r < CG_RANK; ++r) w[r] = live ? __bfloat162float(gw[(size_t)(r0 + r) * a.dim]) : 0.f;
+            __syncthreads();
+        }
         for (int x = tid; x < LC * CG_RANK / 4; x += CG_THREADS) {
             const int t = x / (CG_RANK / 4), q = (x % (CG_RANK / 4)) * 4;
             store4(&in[t][q], t < cnt ? load4_cg(a.decay_in + (size_t)(c * LC + t) * a.ld_decay + r0 + q) : make_float4(0.f, 0.f, 0.f, 0.f));
@@ -361,7 +383,7 @@ __global__ void __launch_bounds__(CG_THREADS) k_channel_decays(RecurrenceArgs a,
     }
     float s = 0.f;
 #pragma unroll
-    for (int x = 0; x < CG_RUN; ++x) { s += channel_log_decay(z[x], a.inv_tau); z[x] = s; }
+    for (int x = 0; x < CG_RUN; ++x) { s += channel_log_decay_fast(z[x], a.inv_tau); z[x] = s; }
     total[run][lane] = s;
     __syncthreads();
     float before = 0.f;
@@ -388,15 +410,18 @@ __device__ __forceinline__ float4 sub4(const float4& a, const float4& b) { retur
 // whole chunk's decay.
 constexpr int LK_THREADS = 512;
 static size_t lk_smem(int mode, int dim, int jt) { return (size_t)LC * ((mode == DECAY_CHANNEL ? 2 : 1) * (dim + 8) + jt + 8) * 2; }
-template <int JT, int MODE>
+// PAIR: two heads that share q and k, one per half of the columns (JT = 128, vdim up to 64); blockIdx.y counts pairs.
+template <int JT, int MODE, bool PAIR>
 __global__ void __launch_bounds__(LK_THREADS, 2) k_chunk_kv(RecurrenceArgs a, float* __restrict__ kv, const float* __restrict__ cum, float* __restrict__ total) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) uint8_t lk_raw[];
-    __shared__ float pw[LC], sL[LC], wsum[LC / 32];             // pw by token: what k is scaled by
+    constexpr int HP = PAIR ? 2 : 1;
+    __shared__ float pws[HP * LC], sL[HP * LC], wsum[HP * LC / 32];             // pws by token: what k is scaled by
     constexpr int VLD = JT + 8, NP = JT / 32;                   // 16-column pairs of tiles per warp
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, head = blockIdx.y, c = blockIdx.x, j0 = blockIdx.z * JT;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, head = blockIdx.y * HP, c = blockIdx.x, j0 = blockIdx.z * JT;
     const int dim = a.dim, vdim = a.vdim, kld = dim + 8, jw = (warp >> 3) * (JT / 2), kvh = head / (a.heads / a.kv_heads);
+    const float* pw = PAIR ? pws + (warp >> 3) * LC : pws;
     bf16* sk = reinterpret_cast<bf16*>(lk_raw);                 // MODE channel: the decayed keys' first terms, then the second
     bf16* sl = sk + LC * kld;
     bf16* sv = MODE == DECAY_CHANNEL ? sl + LC * kld : sl;
@@ -404,15 +429,15 @@ __global__ void __launch_bounds__(LK_THREADS, 2) k_chunk_kv(RecurrenceArgs a, fl
     const size_t row0 = (size_t)c * LC;
     const bf16* kg = reinterpret_cast<const bf16*>(a.k) + row0 * a.ldk + (size_t)kvh * dim;
     const bf16* vg = reinterpret_cast<const bf16*>(a.v) + row0 * a.ldv + (size_t)head * vdim + j0;
-    copy_tile<LK_THREADS, JT / 8>(sv, VLD, vg, a.ldv, LC, cnt, JT, vdim - j0);
+    copy_values<LK_THREADS, JT, PAIR>(sv, vg, a.ldv, LC, cnt, vdim - j0, vdim);
     if (MODE != DECAY_CHANNEL) copy_tile<LK_THREADS, 16>(sk, kld, kg, a.ldk, LC, cnt, dim, dim);
     cp_async_commit();
     if (MODE == DECAY_CONST) {
-        if (tid < LC) pw[tid] = tid < cnt ? a.decay_pow[head * (LC + 1) + cnt - 1 - tid] : 0.f;
+        if (tid < LC) pws[tid] = tid < cnt ? a.decay_pow[head * (LC + 1) + cnt - 1 - tid] : 0.f;
     } else if (MODE == DECAY_HEAD) {
-        head_decays(a, head, row0, cnt, pw, sL, wsum);
-        if (tid < LC) pw[tid] *= exp2f(sL[LC - 1] - sL[tid]);
-        if (tid == 0 && blockIdx.z == 0) total[c * a.heads + head] = sL[LC - 1];
+        head_decays<HP>(a, head, row0, cnt, pws, sL, wsum);
+        if (tid < HP * LC) pws[tid] *= exp2f(sL[tid | (LC - 1)] - sL[tid]);
+        if (tid < HP && blockIdx.z == 0) total[c * a.heads + head + tid] = sL[tid * LC + LC - 1];
     } else {
         const size_t hd = (size_t)a.heads * dim;
         const float* bg = cum + row0 * hd + (size_t)head * dim;
@@ -432,7 +457,8 @@ __global__ void __launch_bounds__(LK_THREADS, 2) k_chunk_kv(RecurrenceArgs a, fl
     cp_async_wait_all();
     __syncthreads();
     const int ksteps = (cnt + 15) / 16;
-    if (j0 + jw >= vdim) return;
+    const int my = PAIR ? head + (warp >> 3) : head, col0 = PAIR ? 0 : j0 + jw;       // this warp's head and its first value column
+    if (col0 >= vdim) return;
     for (int i0 = (warp & 7) * 16; i0 < dim; i0 += 128) {
         float acc[2 * NP][4];
 #pragma unroll
@@ -459,10 +485,10 @@ __global__ void __launch_bounds__(LK_THREADS, 2) k_chunk_kv(RecurrenceArgs a, fl
             mma_row<NP>(acc, ah, b);
             mma_row<NP>(acc, al, b);
         }
-        float* dst = kv + ((size_t)c * a.heads + head) * dim * vdim + (size_t)(i0 + (lane >> 2)) * vdim + j0 + jw + 2 * (lane & 3);
+        float* dst = kv + ((size_t)c * a.heads + my) * dim * vdim + (size_t)(i0 + (lane >> 2)) * vdim + col0 + 2 * (lane & 3);
 #pragma unroll
         for (int nt = 0; nt < 2 * NP; ++nt)
-            if (j0 + jw + nt * 8 < vdim) {
+            if (col0 + nt * 8 < vdim) {
                 *reinterpret_cast<float2*>(dst + nt * 8) = make_float2(acc[nt][0], acc[nt][1]);
                 *reinterpret_cast<float2*>(dst + (size_t)8 * vdim + nt * 8) = make_float2(acc[nt][2], acc[nt][3]);
             }
@@ -516,27 +542,28 @@ __global__ void __launch_bounds__(LN_THREADS) k_chunk_scan(RecurrenceArgs a, con
 }
 
 // ---------------------------------------------------------------- chunked: outputs
-// Rows t0 + lane / 4 (+ 8) of a warp's accumulators -> o
+// Rows t0 + lane / 4 (+ 8) of a warp's accumulators -> columns col0 .. of the head's output.  vrow: the values of row t0 from
+// column col0 on, for the skip.
 template <int NT>
-__device__ __forceinline__ void store_out(const RecurrenceArgs& a, const float (&acc)[NT][4], size_t row0, int cnt, int t0, int head, int j0, int jw, float skip,
-                                          const bf16* sv, int vld) {
+__device__ __forceinline__ void store_out(const RecurrenceArgs& a, const float (&acc)[NT][4], size_t row0, int cnt, int t0, int head, int col0, float skip,
+                                          const bf16* vrow, int vld) {
     const int lane = threadIdx.x & 31;
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
-        const int t = t0 + (lane >> 2) + h * 8;
-        if (t >= cnt) continue;
-        float* orow = a.o + ((row0 + t) * a.heads + head) * a.vdim + j0;
+        const int r = (lane >> 2) + h * 8;
+        if (t0 + r >= cnt) continue;
+        float* orow = a.o + ((row0 + t0 + r) * a.heads + head) * a.vdim;
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt) {
-            const int j = jw + nt * 8 + 2 * (lane & 3);
-            if (j0 + j >= a.vdim) continue;
-            float2 r = make_float2(acc[nt][2 * h] * a.scale, acc[nt][2 * h + 1] * a.scale);
+            const int j = nt * 8 + 2 * (lane & 3);
+            if (col0 + j >= a.vdim) continue;
+            float2 y = make_float2(acc[nt][2 * h] * a.scale, acc[nt][2 * h + 1] * a.scale);
             if (skip != 0.f) {
-                const uint32_t v = lds32(smem_u32(sv + t * vld + j));
-                r.x = fmaf(skip, bf_lo(v), r.x);
-                r.y = fmaf(skip, bf_hi(v), r.y);
+                const uint32_t v = lds32(smem_u32(vrow + r * vld + j));
+                y.x = fmaf(skip, bf_lo(v), y.x);
+                y.y = fmaf(skip, bf_hi(v), y.y);
             }
-            *reinterpret_cast<float2*>(orow + j) = r;
+            *reinterpret_cast<float2*>(orow + col0 + j) = y;
         }
     }
 }
@@ -544,15 +571,18 @@ __device__ __forceinline__ void store_out(const RecurrenceArgs& a, const float (
 // o_t = D(start, t) q_t S + sum over s <= t of (q_t k_s) D(s, t) v_s      (t, s within the chunk; D: decay between two tokens)
 constexpr int LO_THREADS = 512;
 static size_t lo_smem(int dim, int jt) { return ((size_t)2 * LC * (dim + 8) + (size_t)(LC + 2 * dim) * (jt + 8)) * 2; }
-template <int JT, int MODE>
+template <int JT, int MODE, bool PAIR>
 __global__ void __launch_bounds__(LO_THREADS, 1) k_chunk_out(RecurrenceArgs a, const bf16* __restrict__ hi, const bf16* __restrict__ lo) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) uint8_t lo_raw[];
-    __shared__ float pw[LC + 1], sdt[LC], wsum[LC / 32];       // pw: powers of the decay, or (per head and token) running log2 sums
+    constexpr int HP = PAIR ? 2 : 1;
+    __shared__ float pws[HP * LC + 1], sdts[HP * LC], wsum[HP * LC / 32];       // pws: powers of the decay, or (per head and token) running log2 sums
+    __shared__ float ends[MODE == DECAY_HEAD ? HP * LC : 1];                     // step size times the decay up to the end of the token's sixteen
     constexpr int VLD = JT + 8, NP = JT / 32;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, head = blockIdx.y, c = blockIdx.x, j0 = blockIdx.z * JT;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, head = blockIdx.y * HP, c = blockIdx.x, j0 = blockIdx.z * JT;
     const int dim = a.dim, vdim = a.vdim, qld = dim + 8, kvh = head / (a.heads / a.kv_heads);
+    const float *pw = PAIR ? pws + (warp >> 3) * LC : pws, *sdt = PAIR ? sdts + (warp >> 3) * LC : sdts;
     const int cnt = min(LC, a.n - c * LC);
     bf16* sq = reinterpret_cast<bf16*>(lo_raw);
     bf16* sk = sq + LC * qld;
@@ -565,16 +595,17 @@ __global__ void __launch_bounds__(LO_THREADS, 1) k_chunk_out(RecurrenceArgs a, c
     const bf16* vg = reinterpret_cast<const bf16*>(a.v) + row0 * a.ldv + (size_t)head * vdim + j0;
     const size_t plane = ((size_t)c * a.heads + head) * dim * vdim + j0;
     copy_tile<LO_THREADS, 16>(sq, qld, qg, a.ldq, LC, cnt, dim, dim);
-    copy_tile<LO_THREADS, JT / 8>(sh, VLD, hi + plane, vdim, dim, dim, JT, vdim - j0);
-    copy_tile<LO_THREADS, JT / 8>(sl, VLD, lo + plane, vdim, dim, dim, JT, vdim - j0);
+    copy_values<LO_THREADS, JT, PAIR>(sh, hi + plane, vdim, dim, dim, vdim - j0, (size_t)dim * vdim);
+    copy_values<LO_THREADS, JT, PAIR>(sl, lo + plane, vdim, dim, dim, vdim - j0, (size_t)dim * vdim);
     cp_async_commit();
     copy_tile<LO_THREADS, 16>(sk, qld, kg, a.ldk, LC, cnt, dim, dim);
-    copy_tile<LO_THREADS, JT / 8>(sv, VLD, vg, a.ldv, LC, cnt, JT, vdim - j0);
+    copy_values<LO_THREADS, JT, PAIR>(sv, vg, a.ldv, LC, cnt, vdim - j0, vdim);
     cp_async_commit();
     if (MODE == DECAY_CONST)
-        for (int i = tid; i <= LC; i += LO_THREADS) pw[i] = a.decay_pow[head * (LC + 1) + i];
+        for (int i = tid; i <= LC; i += LO_THREADS) pws[i] = a.decay_pow[head * (LC + 1) + i];
     else
-        head_decays(a, head, row0, cnt, sdt, pw, wsum);
+        head_decays<HP>(a, head, row0, cnt, sdts, pws, wsum);
+    if (MODE == DECAY_HEAD && tid < HP * LC) ends[tid] = sdts[tid] * exp2f(pws[tid | 15] - pws[tid]);
     cp_async_wait<1>();
     __syncthreads();
     // the causal work grows with the tokens' place in the chunk: the four warps of a scheduler (warp % 4) take an early and a
@@ -610,7 +641,8 @@ __global__ void __launch_bounds__(LO_THREADS, 1) k_chunk_out(RecurrenceArgs a, c
     for (int nt = 0; nt < 2 * NP; ++nt) { acc[nt][0] *= d0; acc[nt][1] *= d0; acc[nt][2] *= d1; acc[nt][3] *= d1; }
     cp_async_wait<0>();
     __syncthreads();
-    if (t0 >= cnt || j0 + jw >= vdim) return;
+    const int my = PAIR ? head + (warp >> 3) : head, col0 = PAIR ? 0 : j0 + jw;       // this warp's head and its first value column
+    if (t0 >= cnt || col0 >= vdim) return;
     for (int s0 = 0; s0 < t0 + 16; s0 += 32) {         // 32 keys each, up to the diagonal (a last half block is masked)
         float sc[4][4] = {};
         const uint32_t kaddr = smem_u32(sk + (s0 + (lane & 7) + ((lane >> 4) & 1) * 8) * qld + ((lane >> 3) & 1) * 8);
@@ -626,13 +658,25 @@ __global__ void __launch_bounds__(LO_THREADS, 1) k_chunk_out(RecurrenceArgs a, c
             mma16816(sc[3], qa, d[2], d[3]);
         }
 #pragma unroll
-        for (int nt = 0; nt < 4; ++nt)
+        for (int hb = 0; hb < 2; ++hb) {                // sixteen keys each
+            const int kb = s0 + hb * 16;
+            if (MODE == DECAY_HEAD && kb < t0) {        // before this warp's tokens: by way of the sixteen's end
+                const float* f = ends + (pw - pws) + kb;
+                const float f0 = exp2f(l0 - pw[kb + 15]), f1 = exp2f(l1 - pw[kb + 15]);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int ts = s0 + nt * 8 + 2 * (lane & 3) + (e & 1), d = tl + (e >> 1) * 8 - ts;
+                for (int x = 0; x < 8; ++x) {
+                    const int nt = 2 * hb + (x >> 2), e = x & 3;
+                    sc[nt][e] *= (e >> 1 ? f1 : f0) * f[(x >> 2) * 8 + 2 * (lane & 3) + (e & 1)];
+                }
+                continue;
+            }
+#pragma unroll
+            for (int x = 0; x < 8; ++x) {
+                const int nt = 2 * hb + (x >> 2), e = x & 3, ts = s0 + nt * 8 + 2 * (lane & 3) + (e & 1), d = tl + (e >> 1) * 8 - ts;
                 if (MODE == DECAY_CONST) sc[nt][e] = d >= 0 ? sc[nt][e] * pw[d] : 0.f;
                 else sc[nt][e] = d >= 0 ? sc[nt][e] * exp2f((e >> 1 ? l1 : l0) - pw[ts]) * sdt[ts] : 0.f;
             }
+        }
 #pragma unroll
         for (int hb = 0; hb < 2; ++hb) {
             uint32_t b[NP][4];
@@ -647,28 +691,25 @@ __global__ void __launch_bounds__(LO_THREADS, 1) k_chunk_out(RecurrenceArgs a, c
             mma_row<NP>(acc, pl, b);
         }
     }
-    store_out<2 * NP>(a, acc, row0, cnt, t0, head, j0, jw, MODE == DECAY_HEAD ? a.skip[head] : 0.f, sv, VLD);
+    store_out<2 * NP>(a, acc, row0, cnt, t0, my, col0, MODE == DECAY_HEAD ? a.skip[my] : 0.f, sv + t0 * VLD + jw, VLD);
 }
 
 // ---------------------------------------------------------------- chunked: outputs, a decay per key channel
 // The same sums with b_t, the running log2 decays of the chunk (a vector over the key channels).  Sixteen tokens are a block; a
 // warp has one block of queries and half of the columns:
-//   state           (q_t 2^b_t) S
+//   its own block   score by score, sum over the channels of q k 2^(b_t - b_s), the two warps of a block taking half each
 //   earlier blocks  the keys of block j are decayed to that block's end, k_s 2^(b_end(j) - b_s), once for everybody; the queries
 //                   are decayed from the start of their own block and, while the warp walks back over the blocks, by each
 //                   block it passes.  So every factor is a decay over a span of time, at most 1.
-//   its own block   score by score, sum over the channels of q k 2^(b_t - b_s), the two warps of a block taking half each
+//   state           (q_t 2^b_t) S; the state takes the keys' place in shared memory while the values are multiplied
+// STAGED: queries and decays stand in shared memory (dim up to 128), otherwise they are read where they are needed.
 constexpr int BL = 16, NB = LC / BL;
-static size_t co_smem(int dim, int jt) {
+static size_t co_smem(int dim, int jt, bool staged) {
     const size_t states = (size_t)2 * dim * (jt + 8), keys = (size_t)2 * LC * (dim + 8);
-    return ((states > keys ? states : keys) + (size_t)LC * (jt + 8)) * 2 + (size_t)NB * dim * 4 + (size_t)NB * BL * (BL + 2) * 4;
+    return ((states > keys ? states : keys) + (size_t)LC * (jt + 8)) * 2 + (size_t)NB * dim * 4 + (size_t)NB * BL * (BL + 2) * 4 +
+           (staged ? (size_t)LC * (dim + 8) * 6 : 0);
 }
-// bits of two neighbouring queries times 2^(b - ref)
-__device__ __forceinline__ void decay_pair(uint32_t q, const float2& b, const float2& ref, float& x, float& y) {
-    x = bf_lo(q) * exp2f(b.x - ref.x);
-    y = bf_hi(q) * exp2f(b.y - ref.y);
-}
-template <int JT>
+template <int JT, bool STAGED>
 __global__ void __launch_bounds__(LO_THREADS, 1) k_channel_out(RecurrenceArgs a, const bf16* __restrict__ hi, const bf16* __restrict__ lo,
                                                                const float* __restrict__ cum) {
     pdl_trigger();
@@ -681,22 +722,36 @@ __global__ void __launch_bounds__(LO_THREADS, 1) k_channel_out(RecurrenceArgs a,
     float* step = reinterpret_cast<float*>(co_raw);             // [NB][dim]: decay over a whole block
     float* diag = step + NB * dim;                              // [NB][BL][DLD]: scores inside the blocks
     bf16* sv = reinterpret_cast<bf16*>(diag + NB * BL * DLD);   // [LC][VLD]
-    bf16* sh = sv + LC * VLD;                                   // state: first terms [dim][VLD], second terms; later keys: [LC][kld] twice
-    bf16* sl = sh + dim * VLD;
-    bf16 *kh = sh, *kl = sh + LC * kld;
+    bf16* kh = sv + LC * VLD;                                   // keys: first terms (before: as they come) [LC][kld], second terms;
+    bf16* kl = kh + LC * kld;
+    bf16 *sh = kh, *sl = kh + dim * VLD;                        // later the state: first terms [dim][VLD], second terms
+    const int region = max(2 * dim * VLD, 2 * LC * kld);
+    bf16* sq = kh + region;                                     // STAGED: [LC][kld]
+    float* sb = reinterpret_cast<float*>(sq + LC * kld);        // STAGED: [LC][kld]
     const size_t row0 = (size_t)c * LC, hd = (size_t)a.heads * dim;
     const bf16* qg = reinterpret_cast<const bf16*>(a.q) + row0 * a.ldq + (size_t)head * dim;
     const bf16* kg = reinterpret_cast<const bf16*>(a.k) + row0 * a.ldk + (size_t)head * dim;
     const bf16* vg = reinterpret_cast<const bf16*>(a.v) + row0 * a.ldv + (size_t)head * vdim + j0;
     const float* bg = cum + row0 * hd + (size_t)head * dim;
     const size_t plane = ((size_t)c * a.heads + head) * dim * vdim + j0;
-    copy_tile<LO_THREADS, JT / 8>(sh, VLD, hi + plane, vdim, dim, dim, JT, vdim - j0);
-    copy_tile<LO_THREADS, JT / 8>(sl, VLD, lo + plane, vdim, dim, dim, JT, vdim - j0);
+    copy_tile<LO_THREADS, 16>(kh, kld, kg, a.ldk, LC, cnt, dim, dim);
+    if (STAGED) {
+        copy_tile<LO_THREADS, 16>(sq, kld, qg, a.ldq, LC, cnt, dim, dim);
+        for (int t = tid / 32; t < LC; t += LO_THREADS / 32)
+            for (int col = lane * 4; col < dim; col += 128)
+                cp_async16_zfill(sb + t * kld + col, t < cnt ? bg + t * hd + col : bg, t < cnt);
+    }
+    cp_async_commit();
     copy_tile<LO_THREADS, JT / 8>(sv, VLD, vg, a.ldv, LC, cnt, JT, vdim - j0);
     cp_async_commit();
+    // the decays and queries of a row (rows beyond cnt are not asked for)
+    auto brow = [&](int t) { return STAGED ? sb + t * kld : bg + t * hd; };
+    auto qrow = [&](int t) { return STAGED ? sq + t * kld : qg + (size_t)t * a.ldq; };
     const int wr = (warp >> 2) & 1 ? 7 - (warp & 3) : warp & 3, half = warp >> 3, jw = half * (JT / 2);
     const int t0 = wr * BL, tl = t0 + (lane >> 2), dk = dim / 16, c2 = 2 * (lane & 3);
-    const bool on = t0 < cnt;
+    const bool on = t0 < cnt, cols = on && j0 + jw < vdim;
+    cp_async_wait<1>();
+    __syncthreads();
     // ---- scores inside the block: this warp's rows are t0 + 2 x + half, a lane has four channels of every 128
     if (on) {
         float mine[BL];                                         // [s]: this lane's share of rows x = 0 .. 7 after the exchange
@@ -705,27 +760,25 @@ __global__ void __launch_bounds__(LO_THREADS, 1) k_channel_out(RecurrenceArgs a,
         for (int base = 0; base < dim; base += 128) {           // lanes beyond the last channel add zeros
             const int d0 = base + lane * 4;
             const bool ok = d0 < dim;
-            uint2 q[BL / 2];
-            float4 b[BL / 2];
+            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+            float4 q[BL / 2], b[BL / 2];
 #pragma unroll
             for (int x = 0; x < BL / 2; ++x) {
                 const int t = t0 + 2 * x + half;
-                q[x] = make_uint2(0u, 0u);
-                b[x] = make_float4(0.f, 0.f, 0.f, 0.f);
-                if (ok && t < cnt) { q[x] = ld_cg_u2(qg + (size_t)t * a.ldq + d0); b[x] = load4_cg(bg + t * hd + d0); }
+                q[x] = ok && t < cnt ? load4(qrow(t) + d0) : zero;
+                b[x] = ok && t < cnt ? load4(brow(t) + d0) : zero;
             }
 #pragma unroll
             for (int s = 0; s < BL; ++s) {
                 if (t0 + s >= cnt) break;
-                float4 k = make_float4(0.f, 0.f, 0.f, 0.f), e = k;
-                if (ok) { k = load4_cg(kg + (size_t)(t0 + s) * a.ldk + d0); e = load4_cg(bg + (t0 + s) * hd + d0); }
+                const float4 k = ok ? load4(kh + (t0 + s) * kld + d0) : zero, e = ok ? load4(brow(t0 + s) + d0) : zero;
                 float p[BL / 2];
 #pragma unroll
                 for (int x = 0; x < BL / 2; ++x) {
                     p[x] = 0.f;
                     if (2 * x + half >= s && t0 + 2 * x + half < cnt)      // the same for the whole warp
-                        p[x] = bf_lo(q[x].x) * k.x * exp2f(b[x].x - e.x) + bf_hi(q[x].x) * k.y * exp2f(b[x].y - e.y) +
-                               bf_lo(q[x].y) * k.z * exp2f(b[x].z - e.z) + bf_hi(q[x].y) * k.w * exp2f(b[x].w - e.w);
+                        p[x] = q[x].x * k.x * exp2f(b[x].x - e.x) + q[x].y * k.y * exp2f(b[x].y - e.y) + q[x].z * k.z * exp2f(b[x].z - e.z) +
+                               q[x].w * k.w * exp2f(b[x].w - e.w);
                 }
                 // eight sums over the warp: after three exchanges lane l holds row (l & 7) over its group, then the groups meet
 #pragma unroll
@@ -742,90 +795,64 @@ __global__ void __launch_bounds__(LO_THREADS, 1) k_channel_out(RecurrenceArgs a,
                 mine[s] += p[0];
             }
         }
-        if (lane < 8) {                                         // lane l ends with row x = l (bit 2 was decided first)
+        if (lane < 8) {                                         // lane l ends with row x = l
             const int t = 2 * lane + half;
 #pragma unroll
             for (int s = 0; s < BL; ++s) diag[(wr * BL + t) * DLD + s] = s <= t ? mine[s] : 0.f;
         }
     }
-    // ---- state
-    cp_async_wait_all();
     __syncthreads();
-    float acc[2 * NP][4];
-#pragma unroll
-    for (int nt = 0; nt < 2 * NP; ++nt)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) acc[nt][e] = 0.f;
-    // rows beyond the end take the last token's place: their results are not stored
-    const int ra = min(tl, cnt - 1), rb = min(tl + 8, cnt - 1);
-    const float2 zero2 = make_float2(0.f, 0.f);
-    auto load_q = [&](int kk, const float* ref, float (&x)[8]) {        // the A fragment's eight elements, decayed since ref
-        const int col = kk * 16 + c2;
-        const bf16 *qa = qg + (size_t)ra * a.ldq + col, *qb = qg + (size_t)rb * a.ldq + col;
-        const float *ba = bg + ra * hd + col, *bb = bg + rb * hd + col;
-        const float2 r0 = ref ? __ldcg(reinterpret_cast<const float2*>(ref + col)) : zero2, r1 = ref ? __ldcg(reinterpret_cast<const float2*>(ref + col + 8)) : zero2;
-        decay_pair(ld_cg_u32(qa), __ldcg(reinterpret_cast<const float2*>(ba)), r0, x[0], x[1]);
-        decay_pair(ld_cg_u32(qb), __ldcg(reinterpret_cast<const float2*>(bb)), r0, x[2], x[3]);
-        decay_pair(ld_cg_u32(qa + 8), __ldcg(reinterpret_cast<const float2*>(ba + 8)), r1, x[4], x[5]);
-        decay_pair(ld_cg_u32(qb + 8), __ldcg(reinterpret_cast<const float2*>(bb + 8)), r1, x[6], x[7]);
-    };
-    auto split_q = [](const float (&x)[8], uint32_t (&h)[4], uint32_t (&l)[4]) {
-#pragma unroll
-        for (int i = 0; i < 4; ++i) split_pair(x[2 * i], x[2 * i + 1], h[i], l[i]);
-    };
-    const bool cols = j0 + jw < vdim;
-    if (on && cols) {
-#pragma unroll 2
-        for (int kk = 0; kk < dk; ++kk) {
-            float x[8];
-            uint32_t ah[4], al[4], b[NP][4];
-            load_q(kk, nullptr, x);
-            split_q(x, ah, al);
-            const int off = (kk * 16 + (lane & 15)) * VLD + jw + (lane >> 4) * 8;
-#pragma unroll
-            for (int np = 0; np < NP; ++np) ldsm4_t(b[np], smem_u32(sh + off + np * 16));
-            mma_row<NP>(acc, ah, b);
-            mma_row<NP>(acc, al, b);
-#pragma unroll
-            for (int np = 0; np < NP; ++np) ldsm4_t(b[np], smem_u32(sl + off + np * 16));
-            mma_row<NP>(acc, ah, b);
-        }
-    }
-    __syncthreads();
-    // ---- keys decayed to the end of their block, and the blocks' whole decays
+    // ---- keys decayed to the end of their block (in place, with a second term), and the blocks' whole decays
     for (int col = (tid % 16) * 8; col < dim; col += 128)
 #pragma unroll 2
         for (int t = tid / 16; t < LC; t += LO_THREADS / 16) {
             uint4 h = make_uint4(0u, 0u, 0u, 0u), l = h;
             if (t < cnt) {
-                const float* e = bg + (size_t)min(t | (BL - 1), cnt - 1) * hd + col;
-                const float* f = bg + t * hd + col;
-                decay_split8(ld_cg_u4(kg + (size_t)t * a.ldk + col), sub4(load4_cg(e), load4_cg(f)), sub4(load4_cg(e + 4), load4_cg(f + 4)), h, l);
+                const float *e = brow(min(t | (BL - 1), cnt - 1)) + col, *f = brow(t) + col;
+                decay_split8(*reinterpret_cast<const uint4*>(kh + t * kld + col), sub4(load4(e), load4(f)), sub4(load4(e + 4), load4(f + 4)), h, l);
             }
             *reinterpret_cast<uint4*>(kh + t * kld + col) = h;
             *reinterpret_cast<uint4*>(kl + t * kld + col) = l;
         }
-    for (int x = tid; x < NB * dim; x += LO_THREADS) {
-        const int j = x / dim, d = x - j * dim;
-        float s = 0.f;
-        if (j * BL < cnt) s = exp2f(__ldcg(bg + (size_t)min(j * BL + BL - 1, cnt - 1) * hd + d) - (j > 0 ? __ldcg(bg + (size_t)(j * BL - 1) * hd + d) : 0.f));
-        step[x] = s;
-    }
+    for (int j = tid / 64; j < NB; j += LO_THREADS / 64)
+        for (int d = tid & 63; d < dim; d += 64)
+            step[j * dim + d] = j * BL < cnt ? exp2f(brow(min(j * BL + BL - 1, cnt - 1))[d] - (j > 0 ? brow(j * BL - 1)[d] : 0.f)) : 0.f;
+    cp_async_wait_all();
     __syncthreads();
-    if (!on || !cols) return;
+    // rows beyond the end take the last token's place: their results are not stored
+    const int ra = min(tl, cnt - 1), rb = min(tl + 8, cnt - 1);
+    auto load_q = [&](int kk, int ref, float (&x)[8]) {         // the A fragment's eight elements, decayed since token ref (-1: the chunk's start)
+        const int col = kk * 16 + c2;
+        const bf16 *qa = qrow(ra) + col, *qb = qrow(rb) + col;
+        const float *ba = brow(ra) + col, *bb = brow(rb) + col;
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            float2 r = make_float2(0.f, 0.f);
+            if (ref >= 0) r = *reinterpret_cast<const float2*>(brow(ref) + col + 8 * h);
+            const uint32_t u = *reinterpret_cast<const uint32_t*>(qa + 8 * h), v = *reinterpret_cast<const uint32_t*>(qb + 8 * h);
+            const float2 f = *reinterpret_cast<const float2*>(ba + 8 * h), g = *reinterpret_cast<const float2*>(bb + 8 * h);
+            x[4 * h] = bf_lo(u) * exp2f(f.x - r.x);
+            x[4 * h + 1] = bf_hi(u) * exp2f(f.y - r.y);
+            x[4 * h + 2] = bf_lo(v) * exp2f(g.x - r.x);
+            x[4 * h + 3] = bf_hi(v) * exp2f(g.y - r.y);
+        }
+    };
+    auto split_q = [](const float (&x)[8], uint32_t (&h)[4], uint32_t (&l)[4]) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) split_pair(x[2 * i], x[2 * i + 1], h[i], l[i]);
+    };
     // ---- scores against the earlier blocks, block wr - 1 first
     float sc[NB - 1][2][4];
 #pragma unroll
     for (int y = 0; y < NB - 1; ++y)
 #pragma unroll
         for (int e = 0; e < 4; ++e) sc[y][0][e] = sc[y][1][e] = 0.f;
-    if (wr > 0) {
-        const float* ref = bg + (size_t)(t0 - 1) * hd;
+    if (cols && wr > 0) {
         const int koff = ((lane & 7) + ((lane >> 4) & 1) * 8) * kld + ((lane >> 3) & 1) * 8;
 #pragma unroll 1
         for (int kk = 0; kk < dk; ++kk) {
             float x[8];
-            load_q(kk, ref, x);
+            load_q(kk, t0 - 1, x);
 #pragma unroll
             for (int y = 0; y < NB - 1; ++y) {
                 if (y >= wr) break;
@@ -846,6 +873,15 @@ __global__ void __launch_bounds__(LO_THREADS, 1) k_channel_out(RecurrenceArgs a,
             }
         }
     }
+    __syncthreads();                                            // the keys have been read
+    copy_tile<LO_THREADS, JT / 8>(sh, VLD, hi + plane, vdim, dim, dim, JT, vdim - j0);
+    copy_tile<LO_THREADS, JT / 8>(sl, VLD, lo + plane, vdim, dim, dim, JT, vdim - j0);
+    cp_async_commit();
+    float acc[2 * NP][4];
+#pragma unroll
+    for (int nt = 0; nt < 2 * NP; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[nt][e] = 0.f;
     auto add_values = [&](const float (&p0)[4], const float (&p1)[4], int j) {
         uint32_t b[NP][4], ph[4], pl[4];
 #pragma unroll
@@ -857,19 +893,38 @@ __global__ void __launch_bounds__(LO_THREADS, 1) k_channel_out(RecurrenceArgs a,
         mma_row<NP>(acc, ph, b);
         mma_row<NP>(acc, pl, b);
     };
+    if (cols) {
 #pragma unroll
-    for (int y = 0; y < NB - 1; ++y) {
-        if (y >= wr) break;
-        add_values(sc[y][0], sc[y][1], wr - 1 - y);
-    }
-    {
+        for (int y = 0; y < NB - 1; ++y) {
+            if (y >= wr) break;
+            add_values(sc[y][0], sc[y][1], wr - 1 - y);
+        }
         const float* d = diag + (wr * BL + (lane >> 2)) * DLD + c2;
         const float2 u = *reinterpret_cast<const float2*>(d), v = *reinterpret_cast<const float2*>(d + 8 * DLD);
         const float2 w = *reinterpret_cast<const float2*>(d + 8), z = *reinterpret_cast<const float2*>(d + 8 * DLD + 8);
         const float p0[4] = {u.x, u.y, v.x, v.y}, p1[4] = {w.x, w.y, z.x, z.y};
         add_values(p0, p1, wr);
     }
-    store_out<2 * NP>(a, acc, row0, cnt, t0, head, j0, jw, 0.f, sv, VLD);
+    cp_async_wait_all();
+    __syncthreads();
+    if (!cols) return;
+    // ---- state
+#pragma unroll 2
+    for (int kk = 0; kk < dk; ++kk) {
+        float x[8];
+        uint32_t ah[4], al[4], b[NP][4];
+        load_q(kk, -1, x);
+        split_q(x, ah, al);
+        const int off = (kk * 16 + (lane & 15)) * VLD + jw + (lane >> 4) * 8;
+#pragma unroll
+        for (int np = 0; np < NP; ++np) ldsm4_t(b[np], smem_u32(sh + off + np * 16));
+        mma_row<NP>(acc, ah, b);
+        mma_row<NP>(acc, al, b);
+#pragma unroll
+        for (int np = 0; np < NP; ++np) ldsm4_t(b[np], smem_u32(sl + off + np * 16));
+        mma_row<NP>(acc, ah, b);
+    }
+    store_out<2 * NP>(a, acc, row0, cnt, t0, head, j0 + jw, 0.f, sv, VLD);
 }
 
 // ---------------------------------------------------------------- chunked: launches
@@ -878,14 +933,14 @@ size_t recurrence_scratch_bytes(int n, int heads, int dim, int vdim) {
     const size_t chunks = (n + LC - 1) / LC;
     return chunks * heads * ((size_t)dim * vdim * (sizeof(float) + 2 * sizeof(bf16)) + (size_t)LC * dim * 4 + 4);
 }
-static size_t out_smem(int mode, int dim, int jt) { return mode == DECAY_CHANNEL ? co_smem(dim, jt) : lo_smem(dim, jt); }
-static bool tile_fits(int mode, int dim, int jt) { return out_smem(mode, dim, jt) + 2048 <= 232448 && lk_smem(mode, dim, jt) + 2048 <= 232448; }
-// value columns of one CTA: 128 unless the head has no more than 64, or its dim leaves no room for them
-static int column_tile(int mode, int dim, int vdim) { return vdim > 64 && tile_fits(mode, dim, 128) ? 128 : 64; }
+static bool staged(int dim, int jt) { return co_smem(dim, jt, true) + 2048 <= 232448; }
+static size_t out_smem(int mode, int dim, int jt) { return mode == DECAY_CHANNEL ? co_smem(dim, jt, staged(dim, jt)) : lo_smem(dim, jt); }
+static bool tile_fits(int mode, int dim, int jt) { return out_smem(mode, dim, jt) + 4096 <= 232448 && lk_smem(mode, dim, jt) + 4096 <= 232448; }
 bool recurrence_chunked_fits(int mode, int dim) { return tile_fits(mode, dim, 64); }
-template <int JT, int MODE>
+template <int JT, int MODE, bool PAIR>
 static int chunked(Stream& st, const RecurrenceArgs& a) {
-    const int nchunks = (a.n + LC - 1) / LC, jt = (a.vdim + JT - 1) / JT;
+    const int nchunks = (a.n + LC - 1) / LC;
+    const dim3 grid = PAIR ? dim3(nchunks, a.heads / 2) : dim3(nchunks, a.heads, (a.vdim + JT - 1) / JT);
     const size_t elems = (size_t)nchunks * a.heads * a.dim * a.vdim;
     float* kv = reinterpret_cast<float*>(a.scratch);
     bf16 *hi = reinterpret_cast<bf16*>(kv + elems), *lo = hi + elems;
@@ -893,27 +948,34 @@ static int chunked(Stream& st, const RecurrenceArgs& a) {
     float* total = cum + (size_t)nchunks * LC * a.heads * a.dim;                        // [chunks, heads]
     int rc = 0;
     if (MODE == DECAY_CHANNEL) rc = launch(st, k_channel_decays, dim3((a.heads * a.dim + 31) / 32, nchunks), dim3(CG_THREADS), 0, a, cum);
-    if (!rc) rc = allow_smem(k_chunk_kv<JT, MODE>, lk_smem(MODE, a.dim, JT));
-    if (!rc) rc = launch(st, k_chunk_kv<JT, MODE>, dim3(nchunks, a.heads, jt), dim3(LK_THREADS), lk_smem(MODE, a.dim, JT), a, kv, (const float*)cum, total);
+    if (!rc) rc = allow_smem(k_chunk_kv<JT, MODE, PAIR>, lk_smem(MODE, a.dim, JT));
+    if (!rc) rc = launch(st, k_chunk_kv<JT, MODE, PAIR>, grid, dim3(LK_THREADS), lk_smem(MODE, a.dim, JT), a, kv, (const float*)cum, total);
     const size_t quads = (size_t)a.heads * a.dim * a.vdim / 4;
     if (!rc) rc = launch(st, k_chunk_scan<MODE>, dim3((unsigned)((quads + LN_THREADS - 1) / LN_THREADS)), dim3(LN_THREADS), 0, a, (const float*)kv,
                          (const float*)cum, (const float*)total, hi, lo);
     const size_t smem = out_smem(MODE, a.dim, JT);
     if constexpr (MODE == DECAY_CHANNEL) {
-        if (!rc) rc = allow_smem(k_channel_out<JT>, smem);
-        if (!rc) rc = launch(st, k_channel_out<JT>, dim3(nchunks, a.heads, jt), dim3(LO_THREADS), smem, a, (const bf16*)hi, (const bf16*)lo, (const float*)cum);
+        auto go = [&](auto kernel) {
+            const int e = allow_smem(kernel, smem);
+            return e ? e : launch(st, kernel, grid, dim3(LO_THREADS), smem, a, (const bf16*)hi, (const bf16*)lo, (const float*)cum);
+        };
+        if (!rc) rc = staged(a.dim, JT) ? go(k_channel_out<JT, true>) : go(k_channel_out<JT, false>);
     } else {
-        if (!rc) rc = allow_smem(k_chunk_out<JT, MODE>, smem);
-        if (!rc) rc = launch(st, k_chunk_out<JT, MODE>, dim3(nchunks, a.heads, jt), dim3(LO_THREADS), smem, a, (const bf16*)hi, (const bf16*)lo);
+        if (!rc) rc = allow_smem(k_chunk_out<JT, MODE, PAIR>, smem);
+        if (!rc) rc = launch(st, k_chunk_out<JT, MODE, PAIR>, grid, dim3(LO_THREADS), smem, a, (const bf16*)hi, (const bf16*)lo);
     }
     return rc;
 }
 int recurrence_chunked(Stream& st, const RecurrenceArgs& a) {
     if (!recurrence_chunked_fits(a.mode, a.dim) || !a.scratch) return MQ_ERR_UNSUPPORTED;
-    const bool wide = column_tile(a.mode, a.dim, a.vdim) == 128;
-    if (a.mode == DECAY_CONST) return wide ? chunked<128, DECAY_CONST>(st, a) : chunked<64, DECAY_CONST>(st, a);
-    if (a.mode == DECAY_HEAD) return wide ? chunked<128, DECAY_HEAD>(st, a) : chunked<64, DECAY_HEAD>(st, a);
-    return wide ? chunked<128, DECAY_CHANNEL>(st, a) : chunked<64, DECAY_CHANNEL>(st, a);
+    // value columns of one CTA: 128 unless the head has no more than 64, or its dim leaves no room for them
+    const bool roomy = tile_fits(a.mode, a.dim, 128), wide = a.vdim > 64 && roomy;
+    if (a.mode == DECAY_CONST) return wide ? chunked<128, DECAY_CONST, false>(st, a) : chunked<64, DECAY_CONST, false>(st, a);
+    if (a.mode == DECAY_HEAD) {
+        if (wide) return chunked<128, DECAY_HEAD, false>(st, a);
+        return a.vdim <= 64 && roomy && (a.heads / a.kv_heads) % 2 == 0 ? chunked<128, DECAY_HEAD, true>(st, a) : chunked<64, DECAY_HEAD, false>(st, a);
+    }
+    return wide ? chunked<128, DECAY_CHANNEL, false>(st, a) : chunked<64, DECAY_CHANNEL, false>(st, a);
 }
 
 }  // namespace hy

@@ -75,7 +75,7 @@ def feed(dec, ids, portions):
 def check(got, want, dtype, what=""):
     e = vm.errors(got, want)
     print(f"{what} {dtype}: max {float(e.max()):.2e} mean {float(e.mean()):.2e}")
-    assert float(e.max()) <= TOL[dtype], (what, dtype, float(e.max()), int(e.argmax()))
+    assert float(e.max()) <= TOL[dtype] and float(e.mean()) <= TOL[dtype] / 3, (what, dtype, float(e.max()), int(e.argmax()), float(e.mean()))
 
 
 # ---------------------------------------------------------------- whole models
