@@ -63,7 +63,8 @@ enum { ACT_NONE = 0, ACT_SILU = 1, ACT_SWIGLU = 2 };   // SWIGLU: rows 2i, 2i + 
 struct Segment {
     void* out;       // T, or fp32 if f32
     int row0, rows;  // rows without padding; the next segment starts at a multiple of MQH_SEGMENT
-    int ld, act, f32;
+    int ld;
+    short act, f32;
     const float* bias;   // per row, or null; not with SWIGLU
 };
 constexpr int MAX_SEGMENTS = 6;
@@ -124,7 +125,7 @@ struct GatedNorm {
     const void* g;           // T [hv]
     int hv, vp, vd;          // heads * vp; padded and true size of a head
     int parts, part_n;       // part_n elements each
-    int act, gate_first;
+    short act, gate_first;
     float eps;
 };
 // squares are kept per unit of four elements where no part ends inside one, else per element
@@ -142,12 +143,13 @@ template <typename T>
 __device__ __forceinline__ float gate_act(int act, float z) { return act == GATE_SILU ? silu<T>(z) : Elem<T>::sigmoid(z); }
 // One row by a CTA of NW warps.  raw: hv floats, scratch: gated_scratch floats, red: NW floats (all shared); out: T [hv] (may be
 // raw itself for T = float).  w0: the weights of the thread's first two quads, loaded ahead (NW * 128 elements apart).
-template <typename T, int NW>
+// ONE: a single part.
+template <typename T, int NW, bool ONE>
 __device__ __forceinline__ void gated_norm_row(const GatedNorm& a, const float4 (&w0)[2], float* raw, float* scratch, float* red, T* out) {
     constexpr int STRIDE = NW * 128;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const T* gate = reinterpret_cast<const T*>(a.g);
-    const int unit = gated_unit(a), lanes = gated_lanes(a);
+    const int unit = ONE ? 4 : gated_unit(a), lanes = ONE ? 0 : gated_lanes(a);
     float ss = 0.f;
     int n = 0;
     // whole warps go round: lanes beyond the end take part in the exchanges with zeros
@@ -171,7 +173,7 @@ __device__ __forceinline__ void gated_norm_row(const GatedNorm& a, const float4 
             const float4 u = make_float4(v[x].x * s.x, v[x].y * s.y, v[x].z * s.z, v[x].w * s.w);
             const float4 m = a.gate_first ? u : v[x];
             const float4 q = make_float4(m.x * m.x, m.y * m.y, m.z * m.z, m.w * m.w);
-            if (lanes) {
+            if (!ONE && lanes) {
                 float t = q.x + q.y + q.z + q.w;
                 for (int o = lanes >> 1; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
                 const float inv = 1.0f / sqrtf(t / (float)a.part_n + a.eps);
@@ -179,14 +181,14 @@ __device__ __forceinline__ void gated_norm_row(const GatedNorm& a, const float4 
                 continue;
             }
             if (!in) continue;
-            if (a.parts == 1) ss += q.x + q.y + q.z + q.w;
+            if (ONE) ss += q.x + q.y + q.z + q.w;
             else if (unit == 4) scratch[i >> 2] = q.x + q.y + q.z + q.w;
             else store4(scratch + i, q);
             store4(raw + i, make_float4(u.x * w.x, u.y * w.y, u.z * w.z, u.w * w.w));
         }
     }
-    if (lanes) return;
-    if (a.parts == 1) {
+    if (!ONE && lanes) return;
+    if (ONE) {
         const float inv = 1.0f / sqrtf(cta_sum<NW>(ss, red) / (float)a.part_n + a.eps);
         for (int i = tid * 4; i < a.hv; i += STRIDE) {
             const float4 v = load4(raw + i);
@@ -416,21 +418,22 @@ struct AttnDecodeArgs {             // one token at *position
 template <typename T> int attn_decode(Stream& st, const AttnDecodeArgs& a);
 
 // hy_gemv.cu: y = W v for one token, with what the vector is made of and where y goes
-enum { VEC_NORM = 0, VEC_CONCAT = 1, VEC_GATED = 2, VEC_PLAIN = 3, VEC_POST = 4, VEC_POST_NORM = 5 };
+enum { VEC_NORM = 0, VEC_CONCAT = 1, VEC_GATED = 2, VEC_PLAIN = 3, VEC_POST = 4, VEC_POST_NORM = 5, VEC_GATED_PARTS = 6 };
 enum { OUT_SEGMENTS = 0, OUT_ADD = 1, OUT_STORE = 2, OUT_HEAD = 3 };
-struct GemvArgs {
+struct GemvArgs {                   // what every product reads first: its other lines of the parameter bank are fetched behind the wait
     const void* W; int rows, K;
-    // VEC_NORM: rms(x) * gain; VEC_CONCAT: [x; x0], K = 2 width
-    const float* x; const float* x0; const float* gain; float eps; int norm_n;
-    // token != null: x (and x0) is row *token of embed times embed_scale; CTA 0 stores it to x_store / x0_store
-    const int* token; const void* embed; float embed_scale; int vocab; float* x_store; float* x0_store;
-    // VEC_GATED: the first gn.hv elements are the gated norm, the others those of cat; VEC_PLAIN: cat
-    GatedNorm gn; const void* cat;
+    float* y; float mult;           // OUT_ADD: y += mult * (W v); OUT_STORE: y = W v
+    float eps; int norm_n;
+    const void* cat;                // VEC_PLAIN: the vector; VEC_GATED: its elements from gn.hv on
+    const float* x; const float* gain;      // VEC_NORM: rms(x) * gain
+    Segments seg;                   // OUT_SEGMENTS (one row)
+    const float* x0;                // VEC_CONCAT: [x; x0], K = 2 width
     // VEC_POST: x + rms(post_y) * post (post_y null: x); VEC_POST_NORM: the rms norm of that, times gain.  CTA 0 stores the sum
     // to x_store, which must not be x.
     const float* post_y; const float* post;
-    Segments seg;                   // OUT_SEGMENTS (one row)
-    float* y; float mult;           // OUT_ADD: y += mult * (W v); OUT_STORE: y = W v
+    // token != null: x (and x0) is row *token of embed times embed_scale; CTA 0 stores it to x_store / x0_store
+    const int* token; const void* embed; float embed_scale; int vocab; float* x_store; float* x0_store;
+    GatedNorm gn;                   // VEC_GATED (a norm of one part), VEC_GATED_PARTS: the first gn.hv elements
     float* logits; unsigned long long* slot; unsigned int* ticket; int* out_token;   // OUT_HEAD
     unsigned int* status;
 };

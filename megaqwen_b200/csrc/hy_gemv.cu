@@ -23,6 +23,7 @@ namespace mq {
 namespace hy {
 
 constexpr int GV_WARPS = 8, GV_THREADS = GV_WARPS * 32;
+static __host__ __device__ constexpr bool is_gated(int vec) { return vec == VEC_GATED || vec == VEC_GATED_PARTS; }
 
 __device__ __forceinline__ uint4 ld_weight(const void* p) {
     uint4 v;
@@ -44,8 +45,8 @@ constexpr int GV_AHEAD = 2;       // norm weights of the first 2 x 1024 elements
 struct Ahead { float4 gain[GV_AHEAD], post[GV_AHEAD]; };
 template <int VEC>
 __device__ __forceinline__ void fetch_gain(const GemvArgs& a, Ahead& h) {
-    const float* w = VEC == VEC_GATED ? a.gn.w : a.gain;
-    const int n = VEC == VEC_NORM || VEC == VEC_POST_NORM ? a.K : VEC == VEC_GATED ? a.gn.hv : 0;
+    const float* w = is_gated(VEC) ? a.gn.w : a.gain;
+    const int n = VEC == VEC_NORM || VEC == VEC_POST_NORM ? a.K : is_gated(VEC) ? a.gn.hv : 0;
     const int np = (VEC == VEC_POST || VEC == VEC_POST_NORM) && a.post_y ? a.K : 0;
 #pragma unroll
     for (int x = 0; x < GV_AHEAD; ++x) {
@@ -173,12 +174,12 @@ __device__ __forceinline__ void make_vector(const GemvArgs& a, const Ahead& ahea
             }
         }
     } else {
-        const int hv = VEC == VEC_GATED ? a.gn.hv : 0;
+        const int hv = is_gated(VEC) ? a.gn.hv : 0;
         const T* cat = reinterpret_cast<const T*>(a.cat);
         constexpr int E = Elem<T>::PER16;
         for (int i = hv + tid * E; i < K; i += GV_THREADS * E) cp_async16(vec + i, cat + i);
         cp_async_commit();
-        if (VEC == VEC_GATED) gated_norm_row<T, GV_WARPS>(a.gn, ahead.gain, raw, scratch, red, vec);
+        if (is_gated(VEC)) gated_norm_row<T, GV_WARPS, VEC == VEC_GATED>(a.gn, ahead.gain, raw, scratch, red, vec);
         cp_async_wait_all();
     }
 }
@@ -405,7 +406,7 @@ __global__ void __launch_bounds__(GV_THREADS, 2) k_gemv_f32(GemvArgs a) {
 
 // ---------------------------------------------------------------- launches
 template <int VEC>
-static size_t vec_scratch(const GemvArgs& a) { return VEC == VEC_GATED ? (size_t)gated_scratch(a.gn) * 4 : 0; }
+static size_t vec_scratch(const GemvArgs& a) { return is_gated(VEC) ? (size_t)gated_scratch(a.gn) * 4 : 0; }
 template <int VEC, int OUT, bool TALL>
 static int go_mma(Stream& st, const GemvArgs& a) {
     const size_t smem = (size_t)((a.K + 31) / 32) * 64 + (VEC == VEC_CONCAT || VEC == VEC_PLAIN ? 0 : (size_t)a.K * 4) + vec_scratch<VEC>(a);
@@ -436,6 +437,8 @@ int gemv(Stream& st, int vec, int out, const GemvArgs& a) {
     if (vec == VEC_GATED && out == OUT_ADD) return go<VEC_GATED, OUT_ADD>(st, a, t);
     if (vec == VEC_PLAIN && out == OUT_ADD) return go<VEC_PLAIN, OUT_ADD>(st, a, t);
     if (vec == VEC_GATED && out == OUT_STORE) return go<VEC_GATED, OUT_STORE>(st, a, t);
+    if (vec == VEC_GATED_PARTS && out == OUT_ADD) return go<VEC_GATED_PARTS, OUT_ADD>(st, a, t);
+    if (vec == VEC_GATED_PARTS && out == OUT_STORE) return go<VEC_GATED_PARTS, OUT_STORE>(st, a, t);
     if (vec == VEC_PLAIN && out == OUT_STORE) return go<VEC_PLAIN, OUT_STORE>(st, a, t);
     if (vec == VEC_POST && out == OUT_SEGMENTS) return go<VEC_POST, OUT_SEGMENTS>(st, a, t);
     if (vec == VEC_POST_NORM && out == OUT_HEAD) return go<VEC_POST_NORM, OUT_HEAD>(st, a, t);

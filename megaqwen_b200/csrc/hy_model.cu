@@ -154,7 +154,7 @@ static Segments in_segments(const MqhLayer& l, int form, const Work<T>& w) {
     Segments g = {};
     int row = 0;
     auto add = [&](void* out, int rows_, int ld, int act, int f32, const float* bias = nullptr) {
-        g.s[g.n++] = {out, row, rows_, ld, act, f32, bias};
+        g.s[g.n++] = {out, row, rows_, ld, (short)act, (short)f32, bias};
         row += seg_up(rows_);
     };
     const int hd = l.heads * l.dim, hv = hv_of(l), kd = kv_dim(l), h16 = up16(l.heads);
@@ -235,8 +235,8 @@ static RecurrenceArgs recurrence_args(const MqhLayer& l, const Work<T>& w, void*
 }
 template <typename T>
 static GatedNorm gated_args(const MqhLayer& l, const Work<T>& w, float eps) {
-    return {w.o, l.mix_norm, w.g, hv_of(l), l.vdim, l.vdim_n, l.norm_parts, l.mix_norm_n, l.kind == MQH_LIGHTNING ? GATE_SIGMOID : GATE_SILU,
-            l.kind == MQH_MAMBA2, eps};
+    return {w.o, l.mix_norm, w.g, hv_of(l), l.vdim, l.vdim_n, l.norm_parts, l.mix_norm_n,
+            (short)(l.kind == MQH_LIGHTNING ? GATE_SIGMOID : GATE_SILU), (short)(l.kind == MQH_MAMBA2), eps};
 }
 static HeadNorm head_norm(const MqhLayer& l, const float* w, float eps) { return {w, l.mix_norm_n, l.dim, l.rot / 2, eps, l.rope}; }
 // the caches of an attention run: keys, then values, a row per position
@@ -373,7 +373,7 @@ static int mix_one(Stream& st, const MqhModel* m, const MqhLayer& l, const Work<
             r.conv_w = l.conv_w; r.conv_b = l.conv_b; r.taps = l.conv; r.channels = conv_channels(l);
         }
         b.gn = gated_args(l, w, m->eps);
-        *vec = VEC_GATED;
+        *vec = l.norm_parts == 1 ? VEC_GATED : VEC_GATED_PARTS;
         return recurrence_tokens<T>(st, r);
     }
     if (l.kind == MQH_ATTENTION)

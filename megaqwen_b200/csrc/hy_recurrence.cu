@@ -123,7 +123,7 @@ __global__ void __launch_bounds__(RT_THREADS) k_recurrence_tokens(RecurrenceArgs
     constexpr int IPT = CONV ? (2 * MAXI * 32 + 32 + RT_THREADS - 1) / RT_THREADS : 1;  // convolution channels per thread
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, head = blockIdx.y;
     const int j = blockIdx.x * 32 + (tid & 7) * 4, ig = tid >> 3;
-    const int dim = a.dim, vdim = a.vdim, kvh = head / (a.heads / a.kv_heads);
+    const int dim = a.dim, vdim = a.vdim, kvh = MODE == DECAY_HEAD ? head / (a.heads / a.kv_heads) : head;
     float* S = a.state + (size_t)head * dim * vdim;
     const bool live = j < vdim;                     // vdim is a multiple of 16
     float4 s[MAXI];
@@ -134,6 +134,10 @@ __global__ void __launch_bounds__(RT_THREADS) k_recurrence_tokens(RecurrenceArgs
         const int i = ig + 32 * m;
         s[m] = live && i < dim ? load4_cg(S + (size_t)i * vdim + j) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+    const T* q = reinterpret_cast<const T*>(a.q) + (size_t)kvh * dim;
+    const T* k = reinterpret_cast<const T*>(a.k) + (size_t)kvh * dim;
+    const T* v = reinterpret_cast<const T*>(a.v) + (size_t)head * vdim;
+    const size_t ldq = a.ldq, ldk = a.ldk, ldv = a.ldv, ldo = (size_t)a.heads * vdim;
     float decay = 0.f, bias = 0.f, a_neg = 0.f, skip = 0.f;
     if (MODE == DECAY_CONST) decay = a.decay_pow[head * (LC + 1) + 1];
     if (MODE == DECAY_HEAD) { bias = a.dt_bias[head]; a_neg = a.a_neg[head]; skip = a.skip[head]; }
@@ -199,16 +203,12 @@ __global__ void __launch_bounds__(RT_THREADS) k_recurrence_tokens(RecurrenceArgs
         }
         __syncthreads();
     }
-    const T* q = reinterpret_cast<const T*>(a.q) + (size_t)kvh * dim;
-    const T* k = reinterpret_cast<const T*>(a.k) + (size_t)kvh * dim;
-    const T* v = reinterpret_cast<const T*>(a.v) + (size_t)head * vdim;
-    const size_t ldo = (size_t)hv;
     for (int t = 0; t < a.n; ++t) {
         float4 vv = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (live) vv = CONV ? load4(cv + (tid & 7) * 4) : load4_cg(v + (size_t)t * a.ldv + j);
+        if (live) vv = CONV ? load4(cv + (tid & 7) * 4) : load4_cg(v + t * ldv + j);
         float vs = 0.f;                             // the value column whose output this thread stores
         if (MODE == DECAY_HEAD) {
-            if (tid < 32 && blockIdx.x * 32 + tid < vdim) vs = CONV ? cv[tid] : Elem<T>::get(__ldcg(v + (size_t)t * a.ldv + blockIdx.x * 32 + tid));
+            if (tid < 32 && blockIdx.x * 32 + tid < vdim) vs = CONV ? cv[tid] : Elem<T>::get(__ldcg(v + t * ldv + blockIdx.x * 32 + tid));
             const float dt = softplus(__ldcg(a.decay_in + (size_t)t * a.ld_decay + head) + bias);
             decay = expf(a_neg * dt);
             vv.x *= dt; vv.y *= dt; vv.z *= dt; vv.w *= dt;
@@ -241,7 +241,7 @@ __global__ void __launch_bounds__(RT_THREADS) k_recurrence_tokens(RecurrenceArgs
         for (int m = 0; m < MAXI; ++m) {
             const int i = ig + 32 * m;
             if (i >= dim) break;
-            const float ki = CONV ? ck[i] : Elem<T>::get(__ldcg(k + (size_t)t * a.ldk + i)), qi = CONV ? cq[i] : Elem<T>::get(__ldcg(q + (size_t)t * a.ldq + i));
+            const float ki = CONV ? ck[i] : Elem<T>::get(__ldcg(k + t * ldk + i)), qi = CONV ? cq[i] : Elem<T>::get(__ldcg(q + t * ldq + i));
             const float d = MODE == DECAY_CHANNEL ? al[i] : decay;
             s[m].x = fmaf(d, s[m].x, ki * vv.x); s[m].y = fmaf(d, s[m].y, ki * vv.y);
             s[m].z = fmaf(d, s[m].z, ki * vv.z); s[m].w = fmaf(d, s[m].w, ki * vv.w);
@@ -258,7 +258,7 @@ __global__ void __launch_bounds__(RT_THREADS) k_recurrence_tokens(RecurrenceArgs
             float sum = 0.f;
 #pragma unroll
             for (int w = 0; w < 8; ++w) sum += part[w][tid];
-            a.o[t * ldo + (size_t)head * vdim + blockIdx.x * 32 + tid] = MODE == DECAY_HEAD ? fmaf(skip, vs, sum * a.scale) : sum * a.scale;
+            a.o[t * ldo + (size_t)head * vdim + blockIdx.x * 32 + tid] = MODE == DECAY_HEAD ? fmaf(skip, vs, sum) : MODE == DECAY_CHANNEL ? sum * a.scale : sum;
         }
         __syncthreads();
     }

@@ -96,7 +96,7 @@ template int rows<bf16>(Stream&, int, const RowsArgs&);
 template int rows<float>(Stream&, int, const RowsArgs&);
 
 // the gated norm of a mixer's output, row by row
-template <typename T>
+template <typename T, bool ONE>
 __global__ void __launch_bounds__(256) k_gated_norm(GatedNorm a, T* __restrict__ cat, int ldc) {
     pdl_trigger();
     extern __shared__ float gn_raw[];            // [hv], gated_scratch
@@ -111,14 +111,16 @@ __global__ void __launch_bounds__(256) k_gated_norm(GatedNorm a, T* __restrict__
     const size_t r = blockIdx.x;
     a.o += r * a.hv;
     a.g = reinterpret_cast<const T*>(a.g) + r * a.hv;
-    gated_norm_row<T, 8>(a, w0, gn_raw, gn_raw + a.hv, red, cat + r * ldc);
+    gated_norm_row<T, 8, ONE>(a, w0, gn_raw, gn_raw + a.hv, red, cat + r * ldc);
 }
 template <typename T>
 int gated_norm(Stream& st, int n, const GatedNorm& a, T* cat, int ldc) {
     const size_t smem = (size_t)(a.hv + gated_scratch(a)) * 4;
-    const int rc = allow_smem(k_gated_norm<T>, smem);
-    if (rc) return rc;
-    return launch(st, k_gated_norm<T>, dim3(n), dim3(256), smem, a, cat, ldc);
+    auto go = [&](auto kernel) {
+        const int rc = allow_smem(kernel, smem);
+        return rc ? rc : launch(st, kernel, dim3(n), dim3(256), smem, a, cat, ldc);
+    };
+    return a.parts == 1 ? go(k_gated_norm<T, true>) : go(k_gated_norm<T, false>);
 }
 template int gated_norm<bf16>(Stream&, int, const GatedNorm&, bf16*, int);
 template int gated_norm<float>(Stream&, int, const GatedNorm&, float*, int);
