@@ -39,6 +39,29 @@ __device__ __forceinline__ void norm_rotate(const T* src, const HeadNorm& h, con
     __syncwarp();
 }
 
+// The same in registers, a lane with four neighbouring elements, for heads of up to 128 whose rotated halves are whole quads.
+__device__ __forceinline__ bool quad_head(const HeadNorm& h) { return h.dim <= 128 && h.half % 4 == 0; }
+template <typename T>
+__device__ __forceinline__ float4 norm_rotate_quad(const T* src, const HeadNorm& h, const float2* rope) {
+    const int lane = threadIdx.x & 31, i = lane * 4, hq = h.half / 4;
+    const bool in = i < h.dim, low = lane < hq, turns = lane < 2 * hq;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f), w = v, c0 = v, c1 = v;
+    if (in) { v = load4_cg(src + i); w = load4(h.w + i); }
+    if (turns) {
+        const float4* p = reinterpret_cast<const float4*>(rope + (low ? i : i - h.half));
+        c0 = p[0];                                       // cos, sin of two pairs
+        c1 = p[1];
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / (float)h.dim_n + h.eps);
+    v = make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w);
+    const int other = !turns ? lane : low ? lane + hq : lane - hq;
+    const float4 o = make_float4(__shfl_sync(0xffffffffu, v.x, other), __shfl_sync(0xffffffffu, v.y, other), __shfl_sync(0xffffffffu, v.z, other),
+                                 __shfl_sync(0xffffffffu, v.w, other));
+    if (!turns) return v;
+    const float sg = low ? -1.0f : 1.0f;                 // u cos - v sin, v cos + u sin
+    return make_float4(v.x * c0.x + sg * (o.x * c0.y), v.y * c0.z + sg * (o.y * c0.w), v.z * c1.x + sg * (o.z * c1.y), v.w * c1.z + sg * (o.w * c1.w));
+}
+
 // ---------------------------------------------------------------- several tokens
 // One CTA per token, a warp per head: queries in place, keys and values into the caches.
 constexpr int AR_THREADS = 256;
@@ -50,12 +73,22 @@ __global__ void __launch_bounds__(AR_THREADS) k_attn_rows(AttnRowsArgs a) {
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, dim = a.qn.dim;
     const size_t pos = (size_t)a.pos0 + t;
     float* buf = ar_buf + warp * dim;
+    const bool quads = quad_head(a.qn);
     const float2* rope = reinterpret_cast<const float2*>(a.qn.rope) + pos * a.qn.half;
     for (int x = warp; x < a.heads + a.kv_heads; x += AR_THREADS / 32) {
         const bool query = x < a.heads;
         const size_t kc = (pos * a.kv_heads + (x - a.heads)) * dim;
         T* dst = query ? reinterpret_cast<T*>(a.q) + ((size_t)t * a.heads + x) * dim : reinterpret_cast<T*>(a.k_cache) + kc;
         const T* src = query ? dst : reinterpret_cast<const T*>(a.k) + ((size_t)t * a.kv_heads + (x - a.heads)) * dim;
+        if (quads) {
+            const float4 y = norm_rotate_quad(src, query ? a.qn : a.kn, rope);
+            const int i = lane * 4;
+            if (i < dim) {
+                if (!query) store4(reinterpret_cast<T*>(a.v_cache) + kc + i, load4_cg(src + i));
+                store4(dst + i, y);
+            }
+            continue;
+        }
         norm_rotate(src, query ? a.qn : a.kn, rope, buf);
         for (int i = lane * 4; i < dim; i += 128) {
             store4(dst + i, load4(buf + i));
@@ -172,12 +205,19 @@ __global__ void __launch_bounds__(AD_THREADS) k_attn_decode(AttnDecodeArgs a) {
     pdl_wait_cta();
     const float2* rope = reinterpret_cast<const float2*>(a.qn.rope) + (size_t)pc.pos * a.qn.half;
     const bf16* knew = reinterpret_cast<const bf16*>(a.k) + (size_t)g * dim;
+    const bool quads = quad_head(a.qn);
     // query rows 0 .. nh - 1, the new key as row nh; the remaining rows of the product are zeros
     for (int x = warp; x < nh + (has_new ? 1 : 0); x += AD_WARPS) {
         float* b = buf + warp * dim;
         const bool key = x == nh;
         bf16* dst = key ? snew : sq + x * ld;
-        norm_rotate(key ? knew : reinterpret_cast<const bf16*>(a.q) + (size_t)(h0 + x) * dim, key ? a.kn : a.qn, rope, b);
+        const bf16* src = key ? knew : reinterpret_cast<const bf16*>(a.q) + (size_t)(h0 + x) * dim;
+        if (quads) {
+            const float4 y = norm_rotate_quad(src, key ? a.kn : a.qn, rope);
+            if (lane * 4 < dim) store4(b + lane * 4, y);
+        } else {
+            norm_rotate(src, key ? a.kn : a.qn, rope, b);
+        }
         for (int i = lane * 4; i < dim; i += 128) store4(dst + i, load4(b + i));
         if (key)
             for (int i = lane * 4; i < dim; i += 128) {

@@ -100,14 +100,14 @@ struct SegmentSink {
             }
             return;
         }
+        float4 bias[8];                      // asked for side by side
+#pragma unroll
+        for (int q = 0; q < 8; ++q) bias[q] = s.bias && q < nq ? load4(s.bias + c + 4 * q) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
         for (int q = 0; q < 8; ++q) {
             if (q >= nq) break;
-            float4 r = make_float4(__uint_as_float(v[4 * q]), __uint_as_float(v[4 * q + 1]), __uint_as_float(v[4 * q + 2]), __uint_as_float(v[4 * q + 3]));
-            if (s.bias) {
-                const float4 b = load4(s.bias + c + 4 * q);
-                r = make_float4(r.x + b.x, r.y + b.y, r.z + b.z, r.w + b.w);
-            }
+            float4 r = make_float4(__uint_as_float(v[4 * q]) + bias[q].x, __uint_as_float(v[4 * q + 1]) + bias[q].y,
+                                   __uint_as_float(v[4 * q + 2]) + bias[q].z, __uint_as_float(v[4 * q + 3]) + bias[q].w);
             if (s.act == ACT_SILU) r = make_float4(silu<T>(r.x), silu<T>(r.y), silu<T>(r.z), silu<T>(r.w));
             if (s.f32) store4(reinterpret_cast<float*>(s.out) + (size_t)row * s.ld + c + 4 * q, r);
             else store4(reinterpret_cast<T*>(s.out) + (size_t)row * s.ld + c + 4 * q, r);
